@@ -6,8 +6,9 @@ GROUP with storage of its own: one tensor [entries, pages, 2 (K, V), kv_heads, p
 (a flat page of keys then values where the values have another width than the keys, or none), a
 pool of pages and a page table [slots, pages per sequence].  A sequence holds pages only for the
 positions it has (all of them, or a ring that covers its window), so the cache is sized in
-tokens, not in slots x longest sequence.  Entries whose mixers keep a fixed-size state get a
-float32 tensor [slots, *state_shape], zeroed when a slot is taken.
+tokens, not in slots x longest sequence.  Entries whose parts keep fixed-size states get a
+float32 tensor [slots, *state_shape] each, zeroed when a slot is taken; an entry may keep several (told apart by their
+tags) beside its keys and values, and the model itself may keep some (an embedding's).
 
 The library engine has one sequence and one plane per layer and K/V,
 [layer][k|v][max_ctx][kv_dim] (x0ne-core/runtime/src/engine.rs:83-84,191,747-748), and keeps
@@ -99,9 +100,11 @@ class KVGroup:
 class SequenceCache:
     """All groups and state areas of one model, and the slots that index them."""
 
-    def __init__(self, needs: Sequence[CacheNeed], reads_cache_of: Sequence[Optional[int]], capacity_tokens: int,
+    def __init__(self, needs: Sequence, reads_cache_of: Sequence[Optional[int]], capacity_tokens: int,
                  max_seq_len: int, dtype: torch.dtype, device, max_slots: Optional[int] = None,
-                 page_size: int = PAGE_SIZE, max_chunk: int = 1 << 30):
+                 page_size: int = PAGE_SIZE, max_chunk: int = 1 << 30, model_needs: Sequence[CacheNeed] = ()):
+        """`needs`: per run-order entry a CacheNeed, or a list of them (at most one of kind "kv", states with tags of their
+        own); `model_needs`: states that belong to no entry."""
         self.page_size = page_size
         self.device = device
         self.max_seq_len = max_seq_len
@@ -111,20 +114,33 @@ class SequenceCache:
         self.slots = FreeList(self.n_slots, "slot")
         self.lengths = [0] * self.n_slots
         self.groups: List[KVGroup] = []
-        self.states: Dict[int, torch.Tensor] = {}
+        self.states: Dict = {}              # by entry number, or (entry number or None for the model, tag)
         self._group_of: Dict[int, KVGroup] = {}
         self.max_chunk = max_chunk          # most tokens one sequence may bring to one pass
         by_key: Dict[Tuple, List[int]] = {}
-        for e, need in enumerate(needs):
-            if reads_cache_of[e] is not None:
-                continue
-            if need.kind == "kv":
-                by_key.setdefault((need.kv_heads, need.head_dim, need.window, need.v_dim), []).append(e)
-            elif need.kind == "state":
-                self.states[e] = torch.zeros((self.n_slots,) + tuple(need.state_shape), dtype=torch.float32,
-                                             device=device)
-            elif need.kind != "none":
-                raise ValueError(f"run-order entry {e}: unknown cache need {need.kind!r}")
+        kv_needs: Dict[int, CacheNeed] = {}
+        for e, entry_needs in enumerate(needs):
+            for need in ([entry_needs] if isinstance(entry_needs, CacheNeed) else entry_needs):
+                key = self._state_key(e, need.tag)
+                if need.kind == "state":
+                    if key in self.states:
+                        raise ValueError(f"run-order entry {e} keeps two states with the tag {need.tag!r}")
+                    # what a part of the entry keeps is its own, also where the entry reads another entry's keys and values
+                    if need.tag or reads_cache_of[e] is None:
+                        self.states[key] = torch.zeros((self.n_slots,) + tuple(need.state_shape), dtype=torch.float32, device=device)
+                elif need.kind == "kv":
+                    if e in kv_needs:
+                        raise ValueError(f"run-order entry {e} keeps keys and values twice")
+                    kv_needs[e] = need
+                    if reads_cache_of[e] is None:
+                        by_key.setdefault((need.kv_heads, need.head_dim, need.window, need.v_dim), []).append(e)
+                elif need.kind != "none":
+                    raise ValueError(f"run-order entry {e}: unknown cache need {need.kind!r}")
+        for need in model_needs:
+            if need.kind != "state":
+                raise ValueError(f"a model keeps states only, not {need.kind!r}")
+            self.states[self._state_key(None, need.tag)] = torch.zeros((self.n_slots,) + tuple(need.state_shape), dtype=torch.float32,
+                                                                       device=device)
         for (kvh, hd, window, _), entries in by_key.items():
             ring = None
             if window is not None:
@@ -132,7 +148,7 @@ class SequenceCache:
                 # window of the first of them, so the ring must hold window + c - 1 positions.
                 self.max_chunk = min(self.max_chunk, max(page_size, window))
                 ring = min(self.max_seq_pages, pages_for(window + self.max_chunk - 1, page_size) + 1)
-            g = KVGroup(needs[entries[0]], entries, n_pages if window is None else min(n_pages, ring * self.n_slots),
+            g = KVGroup(kv_needs[entries[0]], entries, n_pages if window is None else min(n_pages, ring * self.n_slots),
                         self.n_slots, self.max_seq_pages, ring, page_size, dtype, device)
             self.groups.append(g)
             for e in entries:
@@ -150,8 +166,16 @@ class SequenceCache:
         src = self._reads[entry] if self._reads[entry] is not None else entry
         return self._group_of[src].view(src)
 
-    def state(self, entry: int) -> torch.Tensor:
-        return self.states[entry]
+    @staticmethod
+    def _state_key(entry: Optional[int], tag: str):
+        return (entry, tag) if tag or entry is None else entry
+
+    def state(self, entry: int, tag: str = "") -> torch.Tensor:
+        return self.states[self._state_key(entry, tag)]
+
+    def model_state(self, tag: str) -> torch.Tensor:
+        """A state that belongs to no run-order entry (the previous token an embedding looks at)."""
+        return self.states[self._state_key(None, tag)]
 
     def snapshot_states(self, slots: torch.Tensor):
         """Copies of the fixed-size states of `slots` (a device tensor of slot numbers), to be put back with

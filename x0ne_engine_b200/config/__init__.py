@@ -11,12 +11,15 @@ from .retuvik import ARCHITECTURE as _RETUVIK, MODEL_TYPE as _RETUVIK_TYPE, Retu
 
 from .barorax import ARCHITECTURE as _BARORAX, MODEL_TYPE as _BARORAX_TYPE, BaroraxConfig
 
+from .ravapel import ARCHITECTURE as _RAVAPEL, MODEL_TYPE as _RAVAPEL_TYPE, RavapelConfig
+
 register_architecture(_QWEN3, _QWEN3_TYPE, Qwen3Config)
 register_architecture(_TENETAR, _TENETAR_TYPE, TenetarConfig)
 register_architecture(_ROVURAX, _ROVURAX_TYPE, RovuraxConfig)
 register_architecture(_RETUVIK, _RETUVIK_TYPE, RetuvikConfig)
 register_architecture(_BARORAX, _BARORAX_TYPE, BaroraxConfig)
+register_architecture(_RAVAPEL, _RAVAPEL_TYPE, RavapelConfig)
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "Qwen3Config", "RovuraxConfig", "TenetarConfig", "RetuvikConfig", "BaroraxConfig",
-           "architectures", "config_from_dict", "config_from_folder", "detect",
+           "RavapelConfig",            "architectures", "config_from_dict", "config_from_folder", "detect",
            "register_architecture", "spec_from_folder", "unregister_architecture"]

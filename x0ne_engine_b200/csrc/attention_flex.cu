@@ -3,7 +3,9 @@
 // multiple of 16 in shared memory), values that are the leading part of the key rows (a latent
 // cache read by every head), a chunked mask, a sliding window, first keys that stay visible whatever
 // the window, a per-head sink in the softmax denominator, a per-head slope times the distance i - j taken off the
-// scaled score, a sigmoid gate on the output per (row, head) or per (row, head, value), and results written as float32.
+// scaled score, a sigmoid gate on the output per (row, head) or per (row, head, value), results written as float32, and
+// weights sigmoid(score + a number per head) in the place of the softmax (nothing is normalised over the keys then: the
+// running maximum stays 0 and the sum 1), with results scaled and written to rows wider than the heads.
 //
 // Both kernels are flash attention on `mma.sync` m16n8k16 with float32 accumulation.  Scores,
 // maxima, sums and weights are float32; for the product with the values a weight p is split into
@@ -55,6 +57,10 @@ __device__ __forceinline__ void fx_store(bf16* out, int64_t i, float v, bool f32
     if (f32) reinterpret_cast<float*>(out)[i] = v;
     else out[i] = __float2bfloat16_rn(v);
 }
+
+// sigmoid of x / log2(e), for a score and bias in the exp2 domain; a masked score of minus infinity weighs nothing
+__device__ __forceinline__ float fx_sigmoid2(float x) { return __fdividef(1.0f, 1.0f + exp2f(-x)); }
+__device__ __forceinline__ int64_t fx_out_ld(const AttnExtra& ex, int q_heads, int vd) { return ex.out_ld > 0 ? ex.out_ld : (int64_t)q_heads * vd; }
 
 __device__ __forceinline__ uint32_t fx_pack(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -197,7 +203,7 @@ __device__ __forceinline__ void fx_accumulate(float (*o)[4], const float (*p)[4]
 // ------------------------------------------------------------------------------------------------
 // prefill
 // ------------------------------------------------------------------------------------------------
-template <int DVT>
+template <int DVT, bool SIG>
 __global__ void __launch_bounds__(256, DVT > 16 ? 1 : 2)
 flex_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCache cache, const int32_t* __restrict__ tile_seq,
                     const int32_t* __restrict__ tile_row0, const int32_t* __restrict__ seq_first_row,
@@ -219,6 +225,8 @@ flex_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCac
     const int n_rows = min(FX_TILE_ROWS, seq_first_row[seq + 1] - row0);
     const float sink2 = ex.sink != nullptr ? ex.sink[head] * FX_LOG2E : -INFINITY;
     const bool sloped = ex.slope != nullptr;
+    constexpr bool sig = SIG;
+    const float sb2 = sig ? ex.sig_bias[head] * FX_LOG2E : 0.f;
     const float sl2 = sloped ? ex.slope[head] * FX_LOG2E : 0.f;       // taken off per position of distance, in the exp2 domain
     pdl_wait();
     const int64_t q_ld = ex.q_ld > 0 ? ex.q_ld : (int64_t)q_heads * sh.dk;
@@ -316,6 +324,12 @@ flex_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCac
                 }
             }
         }
+        if (sig) {
+#pragma unroll
+            for (int n = 0; n < 8; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[n][e] = fx_sigmoid2(s[n][e] + sb2);
+        } else {
         mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1));
         mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
         mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1));
@@ -339,6 +353,7 @@ flex_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCac
 #pragma unroll
             for (int n = 0; n < DVT; ++n) { o[n][0] *= al_a; o[n][1] *= al_a; o[n][2] *= al_b; o[n][3] *= al_b; }
         }
+        }
         fx_accumulate<DVT, 4>(o, s, vs, vstride, 0, lane);
         __syncthreads();          // every warp is done with this stage before the page after next is copied into it
     }
@@ -346,7 +361,8 @@ flex_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCac
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 1); l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 1); l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
     float f_a = 1.f, f_b = 1.f;
-    if (ex.sink != nullptr) {
+    if (sig) l_a = l_b = 1.f;
+    else if (ex.sink != nullptr) {
         const float mf_a = fmaxf(m_a, sink2), mf_b = fmaxf(m_b, sink2);
         f_a = exp2f(m_a - mf_a); f_b = exp2f(m_b - mf_b);
         l_a = l_a * f_a + exp2f(sink2 - mf_a);
@@ -354,6 +370,10 @@ flex_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCac
     }
     f_a *= l_a > 0.f ? 1.0f / l_a : 0.f;
     f_b *= l_b > 0.f ? 1.0f / l_b : 0.f;
+    if (ex.out_scale != 0.f) {
+        f_a *= ex.out_scale;
+        f_b *= ex.out_scale;
+    }
     const bool wide = ex.gate != nullptr && ex.gate_wide > 0;       // a gate per value of the head, not one per head
     if (ex.gate != nullptr && !wide) {
         const bf16* gt = (const bf16*)ex.gate;
@@ -362,7 +382,8 @@ flex_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCac
     }
     const bf16* ga = (const bf16*)ex.gate + (int64_t)(row0 + r_a) * ex.gate_ld + (int64_t)head * sh.vd;
     const bf16* gb = (const bf16*)ex.gate + (int64_t)(row0 + r_b) * ex.gate_ld + (int64_t)head * sh.vd;
-    const int64_t oa = ((int64_t)(row0 + r_a) * q_heads + head) * sh.vd, ob = ((int64_t)(row0 + r_b) * q_heads + head) * sh.vd;
+    const int64_t o_ld = fx_out_ld(ex, q_heads, sh.vd);
+    const int64_t oa = (int64_t)(row0 + r_a) * o_ld + ex.out_col + (int64_t)head * sh.vd, ob = (int64_t)(row0 + r_b) * o_ld + ex.out_col + (int64_t)head * sh.vd;
     const bool f32 = ex.out_f32 > 0;
 #pragma unroll
     for (int n = 0; n < DVT; ++n) {
@@ -416,6 +437,8 @@ flex_decode_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCach
     const bool sloped = ex.slope != nullptr;
     const float sl_a = sloped && g < n_items ? ex.slope[head0 + g] * FX_LOG2E : 0.f;
     const float sl_b = sloped && g + 8 < n_items ? ex.slope[head0 + g + 8] * FX_LOG2E : 0.f;
+    const bool sig = ex.sig_bias != nullptr;
+    const float sb_a = sig && g < n_items ? ex.sig_bias[head0 + g] * FX_LOG2E : 0.f, sb_b = sig && g + 8 < n_items ? ex.sig_bias[head0 + g + 8] * FX_LOG2E : 0.f;
     const int key_lo = fx_first_key(pos, window, ex.chunk);
     const int pg_lo = key_lo / FX_PAGE, pg_hi = slot >= 0 ? pos / FX_PAGE : pg_lo - 1;
     // the walk: pages of kept first keys that lie wholly before the window's first page, then the window's pages
@@ -481,6 +504,15 @@ flex_decode_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCach
                 s[n][2 + e] = vis ? sb : -INFINITY;
             }
         }
+        if (sig) {
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    s[n][e] = fx_sigmoid2(s[n][e] + sb_a);
+                    s[n][2 + e] = fx_sigmoid2(s[n][2 + e] + sb_b);
+                }
+        } else {
         float mx_a = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
         float mx_b = fmaxf(fmaxf(s[0][2], s[0][3]), fmaxf(s[1][2], s[1][3]));
         mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1));
@@ -506,11 +538,16 @@ flex_decode_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCach
 #pragma unroll
             for (int n = 0; n < DVT; ++n) { o[n][0] *= al_a; o[n][1] *= al_a; o[n][2] *= al_b; o[n][3] *= al_b; }
         }
+        }
         fx_accumulate<DVT, 1>(o, s, vs, vstride, 16 * warp, lane);
         __syncthreads();
     }
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 1); l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 1); l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
+    if (sig) {          // nothing to weigh the parts against one another by
+        m_a = m_b = 0.f;
+        l_a = l_b = 1.f;
+    }
     // the four warps' results -> shared memory [warp][item][vdp + 2]
     fx_cp_wait<0>();
     __syncthreads();
@@ -549,17 +586,19 @@ flex_decode_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, PagedCach
     if (item >= n_items) return;
     const int head = head0 + item;
     float fin = 1.f;
-    if (ex.sink != nullptr) {
+    if (sig) ll = 1.f;
+    else if (ex.sink != nullptr) {
         const float sink2 = ex.sink[head] * FX_LOG2E;
         const float mf = fmaxf(mm, sink2);
         fin = exp2f(mm - mf);
         ll = ll * fin + exp2f(sink2 - mf);
     }
     fin *= ll > 0.f ? 1.0f / ll : 0.f;
+    if (ex.out_scale != 0.f) fin *= ex.out_scale;
     const bool wide = ex.gate != nullptr && ex.gate_wide > 0;
     if (ex.gate != nullptr && !wide) fin *= 1.0f / (1.0f + expf(-__bfloat162float(((const bf16*)ex.gate)[(int64_t)row * ex.gate_ld + head])));
     const bf16* gw = (const bf16*)ex.gate + (int64_t)row * ex.gate_ld + (int64_t)head * sh.vd;
-    const int64_t orow = ((int64_t)row * q_heads + head) * sh.vd;
+    const int64_t orow = (int64_t)row * fx_out_ld(ex, q_heads, sh.vd) + ex.out_col + (int64_t)head * sh.vd;
     for (int c = c0; c < sh.vd; c += 8) {
         float acc = 0.f;
         for (int w = 0; w < 4; ++w) acc += mg[((int64_t)w * 16 + item) * ps + 2 + c] * f[w];
@@ -601,20 +640,22 @@ flex_decode_merge_kernel(const float* __restrict__ scratch, bf16* __restrict__ o
         if (lane == 0) {
             const int head = head0 + item;
             float fin = 1.f;
-            if (ex.sink != nullptr) {
+            if (ex.sig_bias != nullptr) ll = 1.f;
+            else if (ex.sink != nullptr) {
                 const float sink2 = ex.sink[head] * FX_LOG2E;
                 const float mf = fmaxf(mm, sink2);
                 fin = exp2f(mm - mf);
                 ll = ll * fin + exp2f(sink2 - mf);
             }
             fin *= ll > 0.f ? 1.0f / ll : 0.f;
+            if (ex.out_scale != 0.f) fin *= ex.out_scale;
             if (ex.gate != nullptr && ex.gate_wide <= 0)
                 fin *= 1.0f / (1.0f + expf(-__bfloat162float(((const bf16*)ex.gate)[(int64_t)row * ex.gate_ld + head])));
             fin_s[item] = fin;
         }
     }
     __syncthreads();
-    const int64_t orow = ((int64_t)row * q_heads + head0) * vd;
+    const int64_t orow = (int64_t)row * fx_out_ld(ex, q_heads, vd) + ex.out_col + (int64_t)head0 * vd;
     for (int i = tid; i < n_items * vd; i += 256) {
         const int item = i / vd, c = i - item * vd;
         const float* src = base + (int64_t)item * ps + 2 + c;
@@ -700,11 +741,16 @@ X0NE_API int x0ne_attention_flex_prefill(const void* q, void* out, PagedCache ca
     const size_t smem = fx_prefill_smem(sh, ex.v_from_k > 0);
     X0NE_REQUIRE(smem <= 227 * 1024, "attention_flex: keys of %d need %zu bytes of shared memory", sh.dk, smem);
     const dim3 grid(n_tiles, q_heads), block(256);
-#define FX_PREFILL(DVT)                                                                                                     \
+#define FX_PREFILL_AS(DVT, SIG)                                                                                             \
     do {                                                                                                                    \
-        if (int e = fx_allow_smem(flex_prefill_kernel<DVT>, smem)) return e;                                                \
-        x0ne_launch(flex_prefill_kernel<DVT>, grid, block, smem, stream, (const bf16*)q, (bf16*)out, cache, tile_seq, tile_row0, \
+        if (int e = fx_allow_smem(flex_prefill_kernel<DVT, SIG>, smem)) return e;                                           \
+        x0ne_launch(flex_prefill_kernel<DVT, SIG>, grid, block, smem, stream, (const bf16*)q, (bf16*)out, cache, tile_seq, tile_row0, \
                     seq_first_row, seq_slot, seq_pos0, q_heads, scale, window, ex, sh);                                     \
+    } while (0)
+#define FX_PREFILL(DVT)                                \
+    do {                                               \
+        if (ex.sig_bias != nullptr) FX_PREFILL_AS(DVT, true); \
+        else FX_PREFILL_AS(DVT, false);                \
     } while (0)
     switch (sh.vdp) {
         case 16: FX_PREFILL(2); break;
@@ -717,6 +763,7 @@ X0NE_API int x0ne_attention_flex_prefill(const void* q, void* out, PagedCache ca
         default: FX_PREFILL(32); break;
     }
 #undef FX_PREFILL
+#undef FX_PREFILL_AS
     X0NE_LAUNCH_CHECK();
 }
 

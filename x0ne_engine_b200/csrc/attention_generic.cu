@@ -21,7 +21,8 @@
 // denominator, a sigmoid gate on the output (per (row, head), or per value), a per-head slope times the
 // distance i - j taken off every score, and first keys that stay visible
 // whatever the window (they are taken first, in tiles of 32 from key 0, then the window's), and results written as float32
-// for a caller that goes on in 32-bit.  With none of them asked for the
+// for a caller that goes on in 32-bit; or, instead of the softmax, weights sigmoid(score + a number per head) that nothing
+// normalises, results multiplied by a factor and written to rows wider than the heads.  With none of them asked for the
 // operations and their order are the ones above.
 
 #define ATT_MAX_I 16  // value width <= 32 * ATT_MAX_I
@@ -42,6 +43,7 @@ __global__ void attention_rows_kernel(const T* __restrict__ q, T* __restrict__ o
     const int pos = row_pos[row], slot = row_slot[row];
     float* qs = smem + w * hd;
     const float slope = ex.slope != nullptr ? ex.slope[head] : 0.f;
+    const float sig_b = ex.sig_bias != nullptr ? ex.sig_bias[head] : 0.f;
     const T* qr = q + (int64_t)row * (ex.q_ld > 0 ? ex.q_ld : (int64_t)q_heads * hd) + (int64_t)head * hd;
     for (int d = lane; d < hd; d += 32) qs[d] = to_f32(qr[d]) * scale;
     __syncwarp();
@@ -72,13 +74,18 @@ __global__ void attention_rows_kernel(const T* __restrict__ q, T* __restrict__ o
                 s = ex.slope != nullptr ? a - slope * (float)(pos - j) : a;
             }
         }
-        const float m_new = fmaxf(m, warp_max(s));
-        if (m_new == -INFINITY) continue;  // no readable key in this tile
-        const float p = off >= 0 ? expf(s - m_new) : 0.f;
-        const float alpha = expf(m - m_new);
-        l = l * alpha + warp_sum(p);
+        float p, m_new = m;
+        if (ex.sig_bias != nullptr) {
+            p = off >= 0 ? 1.0f / (1.0f + expf(-(s + sig_b))) : 0.f;
+        } else {
+            m_new = fmaxf(m, warp_max(s));
+            if (m_new == -INFINITY) continue;  // no readable key in this tile
+            p = off >= 0 ? expf(s - m_new) : 0.f;
+            const float alpha = expf(m - m_new);
+            l = l * alpha + warp_sum(p);
 #pragma unroll
-        for (int i = 0; i < ATT_MAX_I; ++i) acc[i] *= alpha;
+            for (int i = 0; i < ATT_MAX_I; ++i) acc[i] *= alpha;
+        }
         const int nt = min(32, j_end - j0 + 1);
         for (int t = 0; t < nt; ++t) {
             const float pt = __shfl_sync(0xffffffffu, p, t);
@@ -96,7 +103,7 @@ __global__ void attention_rows_kernel(const T* __restrict__ q, T* __restrict__ o
         m = m_new;
     }
     }
-    if (ex.sink != nullptr && slot >= 0) {
+    if (ex.sink != nullptr && slot >= 0 && ex.sig_bias == nullptr) {
         const float sk = ex.sink[head];
         const float m_new = fmaxf(m, sk);
         const float alpha = expf(m - m_new);
@@ -104,10 +111,11 @@ __global__ void attention_rows_kernel(const T* __restrict__ q, T* __restrict__ o
 #pragma unroll
         for (int i = 0; i < ATT_MAX_I; ++i) acc[i] *= alpha;
     }
-    const int64_t o0 = ((int64_t)row * q_heads + head) * vd;
+    const int64_t o0 = (int64_t)row * (ex.out_ld > 0 ? ex.out_ld : (int64_t)q_heads * vd) + ex.out_col + (int64_t)head * vd;
     T* o = out + o0;
     float* of = ex.out_f32 > 0 ? reinterpret_cast<float*>(out) + o0 : nullptr;
-    float inv = l > 0.f ? 1.0f / l : 0.f;      // a row with no readable key (a padding row) gets zeros
+    float inv = ex.sig_bias != nullptr ? 1.f : l > 0.f ? 1.0f / l : 0.f;      // a row with no readable key (a padding row) gets zeros
+    if (ex.out_scale != 0.f) inv *= ex.out_scale;
     if (ex.gate != nullptr && ex.gate_wide <= 0) inv *= 1.0f / (1.0f + expf(-to_f32(((const T*)ex.gate)[(int64_t)row * ex.gate_ld + head])));
     const T* gw = ex.gate != nullptr && ex.gate_wide > 0 ? (const T*)ex.gate + (int64_t)row * ex.gate_ld + (int64_t)head * vd : nullptr;
 #pragma unroll

@@ -183,9 +183,11 @@ struct PagedCache {
 __host__ __device__ __forceinline__ int cache_v_dim(const PagedCache& c) { return c.v_dim == 0 ? c.head_dim : (c.v_dim > 0 ? c.v_dim : 0); }
 
 // The gated activation a product's epilogue applies to a (gate, up) pair.  limit <= 0: silu(g) u.  Else the
-// clipped unit: g = min(g, limit), u = clamp(u, -limit, limit), g sigmoid(slope g) (u + shift).
+// clipped unit: g = min(g, limit), u = clamp(u, -limit, limit), g sigmoid(slope g) (u + shift).  `bias`, if given, holds
+// the gate's biases and then the up branch's (float32, one per output each), added before the activation.
 struct GluParams {
     float limit, slope, shift;
+    const float* bias;
 };
 __device__ __forceinline__ float glu_act(float g, float u, const GluParams& p) {
     if (p.limit > 0.f) {
@@ -194,6 +196,15 @@ __device__ __forceinline__ float glu_act(float g, float u, const GluParams& p) {
         return g / (1.0f + expf(-p.slope * g)) * (u + p.shift);
     }
     return g / (1.0f + expf(-g)) * u;
+}
+// the same for output n of N
+__device__ __forceinline__ float glu_act_at(float g, float u, int n, int N, const GluParams& p) {
+    if (p.bias != nullptr) {
+        const int at = n < N ? n : N - 1;
+        g += __ldg(p.bias + at);
+        u += __ldg(p.bias + N + at);
+    }
+    return glu_act(g, u, p);
 }
 
 // What an attention kernel may be asked for beyond causal softmax over a window.  All zero: nothing.
@@ -208,6 +219,10 @@ struct AttnExtra {
     int32_t gate_wide;    // > 0: `gate` holds one value per (row, q head, value) at row * gate_ld + head * value width + value
     const float* slope;   // per q head, or null: slope[h] * (i - j) is taken off the scaled score of query i and key j
     int32_t out_f32;      // > 0: the results are written as float32 whatever the activation type (same places, counted in values)
+    const float* sig_bias;   // per q head, or null: no softmax; key j weighs sigmoid(score + sig_bias[h]), nothing is normalised over keys
+    int64_t out_ld;       // values between consecutive result rows (0: q heads x value width)
+    float out_scale;      // the results are multiplied by it (0: by one)
+    int32_t out_col;      // where the heads start in a result row
 };
 
 // Element offset of (slot, pos, kv head, which = 0 for K / 1 for V); -1 if there is no page, or if

@@ -247,12 +247,13 @@ X0NE_API int x0ne_add_rmsnorm(float* resid, const void* delta, const float* w, v
 // ----------------------------------------------------------------------------------------
 // Residual add of a delta that is normed first, then RMSNorm (a layer with a norm after each
 // sublayer as well as before it):
-//   d = f32(delta) * rsqrt(mean(delta^2) + eps_d) * w_d     (float32, never rounded)
+//   x = f32(delta) + bias_d (null: none);  d = x * rsqrt(mean(x^2) + eps_d) * w_d     (float32, never rounded)
 //   r = resid + d (stored back);  out = T(r * rsqrt(mean(r^2) + eps) * w)
 // Same rows / block conventions as above; both sums of squares are fixed-order block sums.
 // ----------------------------------------------------------------------------------------
 template <typename T>
-__global__ void add_normed_rmsnorm_any_kernel(float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ w_d,
+__global__ void add_normed_rmsnorm_any_kernel(float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ bias_d,
+                                              const float* __restrict__ w_d,
                                               float eps_d, const float* __restrict__ w, T* __restrict__ out,
                                               const int32_t* __restrict__ rows, int hidden, float eps, int keep) {
     extern __shared__ float parked[];
@@ -263,13 +264,13 @@ __global__ void add_normed_rmsnorm_any_kernel(float* __restrict__ resid, const T
     const T* d = delta + src * hidden;
     float dd = 0.f;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-        const float v = to_f32(d[i]);
+        const float v = to_f32(d[i]) + (bias_d != nullptr ? bias_d[i] : 0.f);
         dd = fmaf(v, v, dd);
     }
     const float scale_d = 1.0f / sqrtf(block_reduce(dd, partial, OpSum(), 0.f) / (float)hidden + eps_d);
     float sum_sq = 0.f;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-        const float v = r[i] + to_f32(d[i]) * scale_d * w_d[i];
+        const float v = r[i] + (to_f32(d[i]) + (bias_d != nullptr ? bias_d[i] : 0.f)) * scale_d * w_d[i];
         r[i] = v;
         if (i < keep) parked[i] = v;
         sum_sq = fmaf(v, v, sum_sq);
@@ -284,7 +285,8 @@ __global__ void add_normed_rmsnorm_any_kernel(float* __restrict__ resid, const T
 
 // hidden % 8 == 0 and hidden <= 8 * 1024 * 2: 16-byte accesses, the row and the delta stay in registers.
 template <typename T, int ITS>
-__global__ void __launch_bounds__(1024) add_normed_rmsnorm_vec_kernel(float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ w_d,
+__global__ void __launch_bounds__(1024) add_normed_rmsnorm_vec_kernel(float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ bias_d,
+                                              const float* __restrict__ w_d,
                                               float eps_d, const float* __restrict__ w, T* __restrict__ out,
                                               const int32_t* __restrict__ rows, int hidden, float eps) {
     __shared__ float sh[32];
@@ -302,6 +304,12 @@ __global__ void __launch_bounds__(1024) add_normed_rmsnorm_vec_kernel(float* __r
         if (i < hidden) {
             load8(d + i, dv[it]);
             load8(r + i, v[it]);
+            if (bias_d != nullptr) {
+                float bv[8];
+                load8(bias_d + i, bv);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) dv[it][k] += bv[k];
+            }
 #pragma unroll
             for (int k = 0; k < 8; ++k) dd += dv[it][k] * dv[it][k];
         }
@@ -336,18 +344,18 @@ __global__ void __launch_bounds__(1024) add_normed_rmsnorm_vec_kernel(float* __r
     }
 }
 
-X0NE_API int x0ne_add_normed_rmsnorm(float* resid, const void* delta, const float* w_d, float eps_d, const float* w, void* out,
+X0NE_API int x0ne_add_normed_rmsnorm(float* resid, const void* delta, const float* bias_d, const float* w_d, float eps_d, const float* w, void* out,
                                      int dt, const int32_t* rows, int n_rows, int hidden, float eps, cudaStream_t stream) {
     X0NE_REQUIRE(n_rows >= 0 && hidden > 0 && delta != nullptr && w_d != nullptr, "add_normed_rmsnorm: rows %d hidden %d", n_rows, hidden);
     X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "add_normed_rmsnorm: unknown dtype tag %d", dt);
     if (n_rows == 0) return 0;
     if (hidden % 8 == 0 && hidden <= 8 * 1024 * 2 &&
-        ((((uintptr_t)resid | (uintptr_t)delta | (uintptr_t)w_d | (uintptr_t)w | (uintptr_t)out) & 15) == 0)) {
+        ((((uintptr_t)resid | (uintptr_t)delta | (uintptr_t)bias_d | (uintptr_t)w_d | (uintptr_t)w | (uintptr_t)out) & 15) == 0)) {
         int threads = (hidden / 8 + 31) / 32 * 32;
         if (threads > 1024) threads = 1024;
         if (hidden / 8 > 512 && hidden / 8 <= 1024) threads = 512;
         const int sweeps = (hidden / 8 + threads - 1) / threads;
-#define X0NE_ANR(T, ITS) x0ne_launch(add_normed_rmsnorm_vec_kernel<T, ITS>, dim3(n_rows), dim3(threads), 0, stream, resid, (const T*)delta, w_d, eps_d, w, (T*)out, rows, hidden, eps)
+#define X0NE_ANR(T, ITS) x0ne_launch(add_normed_rmsnorm_vec_kernel<T, ITS>, dim3(n_rows), dim3(threads), 0, stream, resid, (const T*)delta, bias_d, w_d, eps_d, w, (T*)out, rows, hidden, eps)
         if (dt == X0NE_F32) {
             if (sweeps <= 1) X0NE_ANR(float, 1); else X0NE_ANR(float, 2);
         } else {
@@ -359,9 +367,9 @@ X0NE_API int x0ne_add_normed_rmsnorm(float* resid, const void* delta, const floa
     const int keep = hidden <= 10240 ? hidden : 0;
     const size_t smem = (size_t)keep * sizeof(float);
     if (dt == X0NE_F32)
-        x0ne_launch(add_normed_rmsnorm_any_kernel<float>, dim3(n_rows), dim3(256), smem, stream, resid, (const float*)delta, w_d, eps_d, w, (float*)out, rows, hidden, eps, keep);
+        x0ne_launch(add_normed_rmsnorm_any_kernel<float>, dim3(n_rows), dim3(256), smem, stream, resid, (const float*)delta, bias_d, w_d, eps_d, w, (float*)out, rows, hidden, eps, keep);
     else
-        x0ne_launch(add_normed_rmsnorm_any_kernel<bf16>, dim3(n_rows), dim3(256), smem, stream, resid, (const bf16*)delta, w_d, eps_d, w, (bf16*)out, rows, hidden, eps, keep);
+        x0ne_launch(add_normed_rmsnorm_any_kernel<bf16>, dim3(n_rows), dim3(256), smem, stream, resid, (const bf16*)delta, bias_d, w_d, eps_d, w, (bf16*)out, rows, hidden, eps, keep);
     X0NE_LAUNCH_CHECK();
 }
 
@@ -663,22 +671,26 @@ X0NE_API int x0ne_qk_norm_rope_kv_write(const void* qkv, int dt, const float* no
 }
 
 // ----------------------------------------------------------------------------------------
-// SwiGLU on the packed [gate; up] row: out[i] = T(g / (1 + expf(-g)) * u)
-// (x0ne-core/kernels/cuda/swiglu.cu:5-11).
+// SwiGLU on the packed [gate; up] row: out[i] = T(g / (1 + expf(-g)) * u), g and u with `bias` (packed alike,
+// float32) added first if it is given (x0ne-core/kernels/cuda/swiglu.cu:5-11).
 // ----------------------------------------------------------------------------------------
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter) {
+__global__ void swiglu_kernel(const T* __restrict__ gate_up, const float* __restrict__ bias, T* __restrict__ out, int inter) {
     pdl_prologue();
     const int i = blockIdx.x * blockDim.x + threadIdx.x, r = blockIdx.y;
     if (i >= inter) return;
     const T* row = gate_up + (int64_t)r * 2 * inter;
-    const float g = to_f32(row[i]), u = to_f32(row[inter + i]);
+    float g = to_f32(row[i]), u = to_f32(row[inter + i]);
+    if (bias != nullptr) {
+        g += bias[i];
+        u += bias[inter + i];
+    }
     out[(int64_t)r * inter + i] = from_f32<T>(g / (1.0f + expf(-g)) * u);
 }
 
 // 8 values per thread with 16-byte accesses (inter % 8 == 0 and aligned rows).
 template <typename T>
-__global__ void swiglu_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, int64_t total8) {
+__global__ void swiglu_vec_kernel(const T* __restrict__ gate_up, const float* __restrict__ bias, T* __restrict__ out, int inter, int64_t total8) {
     pdl_prologue();
     const int per_row = inter / 8;
     for (int64_t e = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; e < total8; e += (int64_t)gridDim.x * blockDim.x) {
@@ -688,25 +700,32 @@ __global__ void swiglu_vec_kernel(const T* __restrict__ gate_up, T* __restrict__
         float g[8], u[8], o[8];
         load8(row + i, g);
         load8(row + inter + i, u);
+        if (bias != nullptr) {
+            float b[8], c[8];
+            load8(bias + i, b);
+            load8(bias + inter + i, c);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) { g[k] += b[k]; u[k] += c[k]; }
+        }
 #pragma unroll
         for (int k = 0; k < 8; ++k) o[k] = g[k] / (1.0f + expf(-g[k])) * u[k];
         store8(out + r * inter + i, o);
     }
 }
 
-X0NE_API int x0ne_swiglu(const void* gate_up, void* out, int dt, int n_rows, int inter, cudaStream_t stream) {
+X0NE_API int x0ne_swiglu(const void* gate_up, const float* bias, void* out, int dt, int n_rows, int inter, cudaStream_t stream) {
     X0NE_REQUIRE(n_rows >= 0 && inter > 0, "swiglu: rows %d inter %d", n_rows, inter);
     if (n_rows == 0) return 0;
     X0NE_REQUIRE(n_rows <= 65535 * 1024, "swiglu: too many rows for one launch");
     const int esize = dt == X0NE_F32 ? 4 : 2;
-    if (inter % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0 && ((int64_t)inter * esize) % 16 == 0) {
+    if (inter % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)bias | (uintptr_t)out) & 15) == 0 && ((int64_t)inter * esize) % 16 == 0) {
         const int64_t total8 = (int64_t)n_rows * (inter / 8);
         int64_t blocks = (total8 + 255) / 256;
         if (blocks > 148 * 16) blocks = 148 * 16;
         if (dt == X0NE_F32)
-            x0ne_launch(swiglu_vec_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, inter, total8);
+            x0ne_launch(swiglu_vec_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)gate_up, bias, (float*)out, inter, total8);
         else if (dt == X0NE_BF16)
-            x0ne_launch(swiglu_vec_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, inter, total8);
+            x0ne_launch(swiglu_vec_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, stream, (const bf16*)gate_up, bias, (bf16*)out, inter, total8);
         else
             X0NE_REQUIRE(false, "swiglu: unknown dtype tag %d", dt);
         X0NE_LAUNCH_CHECK();
@@ -715,10 +734,10 @@ X0NE_API int x0ne_swiglu(const void* gate_up, void* out, int dt, int n_rows, int
         const int nr = n_rows - r0 < 65535 ? n_rows - r0 : 65535;
         dim3 grid((inter + 255) / 256, nr);
         if (dt == X0NE_F32)
-            x0ne_launch(swiglu_kernel<float>, dim3(grid), dim3(256), 0, stream, (const float*)gate_up + (int64_t)r0 * 2 * inter,
+            x0ne_launch(swiglu_kernel<float>, dim3(grid), dim3(256), 0, stream, (const float*)gate_up + (int64_t)r0 * 2 * inter, bias,
                         (float*)out + (int64_t)r0 * inter, inter);
         else if (dt == X0NE_BF16)
-            x0ne_launch(swiglu_kernel<bf16>, dim3(grid), dim3(256), 0, stream, (const bf16*)gate_up + (int64_t)r0 * 2 * inter,
+            x0ne_launch(swiglu_kernel<bf16>, dim3(grid), dim3(256), 0, stream, (const bf16*)gate_up + (int64_t)r0 * 2 * inter, bias,
                         (bf16*)out + (int64_t)r0 * inter, inter);
         else
             X0NE_REQUIRE(false, "swiglu: unknown dtype tag %d", dt);
@@ -837,5 +856,177 @@ X0NE_API int x0ne_open_pass(float* resid, const void* delta, int dt, const void*
     else if (table_dt == X0NE_F32) X0NE_OPEN(bf16, float);
     else X0NE_OPEN(bf16, bf16);
 #undef X0NE_OPEN
+    X0NE_LAUNCH_CHECK();
+}
+
+// ----------------------------------------------------------------------------------------
+// Embedding as a sum of up to three rows, added in float32 in this order:
+//   table[token] + pairs[(prev * mul_prev + token * mul_cur) mod buckets] + positions[pos]
+// The pair row of a sequence's first token (pos 0) is number `buckets`, the last one.  The token before a row is the row
+// above's where that continues the same sequence in this pass, else the one the sequence's state keeps; the block of the
+// first row a sequence brings reads that and leaves the sequence's last token of the pass there (one int32 per slot,
+// `state_stride` apart; no other block touches it).  `pairs` and `positions` may be null; `copy`, if given, receives the
+// rows too (what later stages of the model call the embedding output).
+// ----------------------------------------------------------------------------------------
+struct EmbedSumArgs {
+    const void* table;
+    const void* pairs;
+    const void* positions;
+    const int32_t* tokens;
+    const int32_t* row_slot;
+    const int32_t* row_pos;
+    const int32_t* seq_first_row;
+    int32_t* last_token;            // per slot (null without `pairs`)
+    int64_t state_stride;
+    float* resid;
+    float* copy;
+    int64_t mul_prev, mul_cur, buckets;
+    int32_t n_seqs, hidden, vocab, n_positions;
+};
+
+template <typename T, bool VEC>
+__global__ void embed_sum_kernel(EmbedSumArgs a) {
+    __shared__ int prev_s;
+    pdl_prologue();
+    const int row = blockIdx.x, slot = a.row_slot[row], pos = a.row_pos[row], t = a.tokens[row];
+    int64_t pair = a.buckets;
+    if (a.pairs != nullptr) {
+        const bool above = row > 0 && slot >= 0 && a.row_slot[row - 1] == slot && a.row_pos[row - 1] == pos - 1;
+        int prev = 0;
+        if (above) {
+            prev = a.tokens[row - 1];
+        } else if (slot >= 0) {             // (the same for every thread of the block)
+            if (threadIdx.x == 0) {
+                int32_t* kept = a.last_token + (int64_t)slot * a.state_stride;
+                prev_s = *kept;
+                int lo = 0, hi = a.n_seqs - 1;          // the sequence whose first row this is: first rows ascend
+                while (lo < hi) {
+                    const int mid = (lo + hi + 1) / 2;
+                    if (a.seq_first_row[mid] <= row) lo = mid; else hi = mid - 1;
+                }
+                *kept = a.tokens[a.seq_first_row[lo + 1] - 1];
+            }
+            __syncthreads();
+            prev = prev_s;
+        }
+        if (pos > 0) {
+            int64_t b = ((int64_t)prev * a.mul_prev + (int64_t)t * a.mul_cur) % a.buckets;
+            pair = b < 0 ? b + a.buckets : b;
+        }
+    }
+    const bool none = t < 0 || t >= a.vocab;
+    const T* e = (const T*)a.table + (int64_t)(none ? 0 : t) * a.hidden;
+    const T* g = a.pairs != nullptr ? (const T*)a.pairs + pair * a.hidden : nullptr;
+    const T* p = a.positions != nullptr && pos >= 0 && pos < a.n_positions ? (const T*)a.positions + (int64_t)pos * a.hidden : nullptr;
+    float* dst = a.resid + (int64_t)row * a.hidden;
+    float* cp = a.copy != nullptr ? a.copy + (int64_t)row * a.hidden : nullptr;
+    if (VEC) {
+        for (int i = threadIdx.x * 8; i < a.hidden; i += blockDim.x * 8) {
+            float v[8], x[8], y[8];
+            load8(e + i, v);
+            if (g != nullptr) load8(g + i, x);
+            if (p != nullptr) load8(p + i, y);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) {
+                if (none) v[k] = 0.f;
+                if (g != nullptr) v[k] += x[k];
+                if (p != nullptr) v[k] += y[k];
+            }
+            store8(dst + i, v);
+            if (cp != nullptr) store8(cp + i, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < a.hidden; i += blockDim.x) {
+            float v = none ? 0.f : to_f32(e[i]);
+            if (g != nullptr) v += to_f32(g[i]);
+            if (p != nullptr) v += to_f32(p[i]);
+            dst[i] = v;
+            if (cp != nullptr) cp[i] = v;
+        }
+    }
+}
+
+X0NE_API int x0ne_embed_sum(EmbedSumArgs a, int dt, int n_rows, cudaStream_t stream) {
+    X0NE_REQUIRE(n_rows >= 0 && a.hidden > 0 && a.vocab > 0 && a.n_seqs >= 0, "embed_sum: rows %d hidden %d vocab %d", n_rows, a.hidden, a.vocab);
+    X0NE_REQUIRE(a.pairs == nullptr || (a.buckets > 0 && a.last_token != nullptr && a.seq_first_row != nullptr && a.n_seqs > 0), "embed_sum: pair rows need buckets, the sequences' last tokens and their rows");
+    X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "embed_sum: unknown dtype tag %d", dt);
+    if (n_rows == 0) return 0;
+    const bool vec = a.hidden % 8 == 0 && (((uintptr_t)a.table | (uintptr_t)a.pairs | (uintptr_t)a.positions | (uintptr_t)a.resid | (uintptr_t)a.copy) & 15) == 0;
+    const int work = vec ? a.hidden / 8 : a.hidden;
+    const int threads = work >= 256 ? 256 : (work + 31) / 32 * 32;
+#define X0NE_ES(T, V) x0ne_launch(embed_sum_kernel<T, V>, dim3(n_rows), dim3(threads), 0, stream, a)
+    if (dt == X0NE_F32) { if (vec) X0NE_ES(float, true); else X0NE_ES(float, false); }
+    else { if (vec) X0NE_ES(bf16, true); else X0NE_ES(bf16, false); }
+#undef X0NE_ES
+    X0NE_LAUNCH_CHECK();
+}
+
+// ----------------------------------------------------------------------------------------
+// The operand of a product over two concatenated rows:  out[r] = [ x | x0[r] ]  with
+//   x = resid[r] + norm(delta[r] + bias_d) * w_d      (delta null: resid alone; w_d null: delta added as it is)
+// in float32, rounded once to the activation type.  The residual is only read.  With `lo` (bfloat16 runs) the rows n_rows
+// .. 2 n_rows - 1 of out receive what that rounding lost, rounded in turn: the product over both, added up, sees the
+// float32 values to 16 bits.
+// One block per row; the sum of squares is a fixed-order block sum.
+// ----------------------------------------------------------------------------------------
+template <typename T>
+__global__ void concat_rows_kernel(const float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ bias_d,
+                                   const float* __restrict__ w_d, float eps_d, const float* __restrict__ x0, T* __restrict__ out, int n_rows,
+                                   int hidden, int lo) {
+    __shared__ float sh[32];
+    pdl_prologue();
+    const int64_t row = blockIdx.x;
+    const float* r = resid + row * hidden;
+    const float* z = x0 + row * hidden;
+    const T* d = delta != nullptr ? delta + row * hidden : nullptr;
+    T* o = out + row * 2 * hidden;
+    T* l = lo ? out + (row + n_rows) * 2 * hidden : nullptr;
+    float scale = 1.f;
+    if (d != nullptr && w_d != nullptr) {
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+            const float v = to_f32(d[i]) + (bias_d != nullptr ? bias_d[i] : 0.f);
+            ss = fmaf(v, v, ss);
+        }
+        scale = 1.0f / sqrtf(block_sum(ss, sh) / (float)hidden + eps_d);
+    }
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        float v = r[i];
+        if (d != nullptr) v += (to_f32(d[i]) + (bias_d != nullptr ? bias_d[i] : 0.f)) * scale * (w_d != nullptr ? w_d[i] : 1.f);
+        const float w = z[i];
+        const T hv = from_f32<T>(v), hw = from_f32<T>(w);
+        o[i] = hv;
+        o[hidden + i] = hw;
+        if (l != nullptr) {
+            l[i] = from_f32<T>(v - to_f32(hv));
+            l[hidden + i] = from_f32<T>(w - to_f32(hw));
+        }
+    }
+}
+
+// out[i] = a[i] + b[i], float32 (the two halves of such a product)
+__global__ void add_f32_kernel(const float* __restrict__ a, const float* __restrict__ b, float* __restrict__ out, int64_t total) {
+    pdl_prologue();
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) out[i] = a[i] + b[i];
+}
+
+X0NE_API int x0ne_concat_rows(const float* resid, const void* delta, int dt, const float* bias_d, const float* w_d, float eps_d, const float* x0,
+                              void* out, int n_rows, int hidden, int lo, cudaStream_t stream) {
+    X0NE_REQUIRE(n_rows >= 0 && hidden > 0 && resid != nullptr && x0 != nullptr && out != nullptr, "concat_rows: rows %d hidden %d", n_rows, hidden);
+    X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "concat_rows: unknown dtype tag %d", dt);
+    if (n_rows == 0) return 0;
+    const int block = hidden >= 512 ? 512 : (hidden + 31) / 32 * 32;
+    if (dt == X0NE_F32)
+        x0ne_launch(concat_rows_kernel<float>, dim3(n_rows), dim3(block), 0, stream, resid, (const float*)delta, bias_d, w_d, eps_d, x0, (float*)out, n_rows, hidden, lo);
+    else
+        x0ne_launch(concat_rows_kernel<bf16>, dim3(n_rows), dim3(block), 0, stream, resid, (const bf16*)delta, bias_d, w_d, eps_d, x0, (bf16*)out, n_rows, hidden, lo);
+    X0NE_LAUNCH_CHECK();
+}
+
+X0NE_API int x0ne_add_f32(const float* a, const float* b, float* out, int64_t total, cudaStream_t stream) {
+    X0NE_REQUIRE(total >= 0 && a != nullptr && b != nullptr && out != nullptr, "add_f32: %lld values", (long long)total);
+    if (total == 0) return 0;
+    const int64_t blocks = (total + 255) / 256;
+    x0ne_launch(add_f32_kernel, dim3((unsigned)(blocks < 148 * 64 ? blocks : 148 * 64)), dim3(256), 0, stream, a, b, out, total);
     X0NE_LAUNCH_CHECK();
 }

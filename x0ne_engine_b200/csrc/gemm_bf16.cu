@@ -178,7 +178,7 @@ __global__ void __launch_bounds__(SM_WARPS * 32) gemm_smallm_kernel(const bf16* 
             }
             if (n < N && m < M) {
                 float out = v[0];
-                if (SWIGLU) out = glu_act(v[0], v[SETS - 1], glu);
+                if (SWIGLU) out = glu_act_at(v[0], v[SETS - 1], n, N, glu);
                 Y[(int64_t)m * ldy + n] = from_f32<OutT>(out);
             }
         }
@@ -221,10 +221,10 @@ static int launch_smallm(const bf16* W, const bf16* X, OutT* Y, int M, int N, in
 
 // out_kind: 0 = bfloat16, 1 = float32, 2 = bfloat16 with SwiGLU over the packed [gate; up] weight
 // (W then has 2*N rows and y has N columns).
-// With out_kind 2, (limit, slope, shift) choose the gated activation (`GluParams`; limit 0: SwiGLU).
+// With out_kind 2, (limit, slope, shift, bias) choose the gated activation (`GluParams`; limit 0: SwiGLU; bias may be null).
 X0NE_API int x0ne_gemm_bf16_smallm_glu(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,
-                                       int sms, float limit, float slope, float shift, cudaStream_t stream) {
-    const GluParams glu = {limit, slope, shift};
+                                       int sms, float limit, float slope, float shift, const float* bias, cudaStream_t stream) {
+    const GluParams glu = {limit, slope, shift, bias};
     X0NE_REQUIRE(M >= 0 && M <= 32 && N > 0 && K > 0, "gemm_smallm: M %d (at most 32) N %d K %d", M, N, K);
     X0NE_REQUIRE(K % 8 == 0, "gemm_smallm: K %d is not a multiple of 8", K);
     X0NE_REQUIRE(ldy >= N && sms > 0 && out_kind >= 0 && out_kind <= 2, "gemm_smallm: ldy %d N %d kind %d", ldy, N, out_kind);
@@ -245,5 +245,5 @@ X0NE_API int x0ne_gemm_bf16_smallm_glu(const void* W, const void* X, void* Y, in
 
 X0NE_API int x0ne_gemm_bf16_smallm(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,
                                    int sms, cudaStream_t stream) {
-    return x0ne_gemm_bf16_smallm_glu(W, X, Y, M, N, K, ldy, out_kind, sms, 0.f, 0.f, 0.f, stream);
+    return x0ne_gemm_bf16_smallm_glu(W, X, Y, M, N, K, ldy, out_kind, sms, 0.f, 0.f, 0.f, nullptr, stream);
 }

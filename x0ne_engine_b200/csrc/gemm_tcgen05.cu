@@ -167,7 +167,7 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_kernel(const __grid_consta
                     float u[32];
                     tc_ld32(trow + 128 + c * 32, u);
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = glu_act(v[i], u[i], glu);
+                    for (int i = 0; i < 32; ++i) v[i] = glu_act_at(v[i], u[i], n0 + c * 32 + i, N, glu);
                 }
                 const int n = n0 + c * 32;
                 if (m < M) {
@@ -367,7 +367,7 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_pair_kernel(const __grid_c
                     float u[32];
                     tc_ld32(trow + 128 + c * 32, u);
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = glu_act(v[i], u[i], glu);
+                    for (int i = 0; i < 32; ++i) v[i] = glu_act_at(v[i], u[i], n0 + c * 32 + i, N, glu);
                 }
                 const int n = n0 + c * 32;
                 if (m < M) {
@@ -502,10 +502,10 @@ static int launch_tc_pair(const void* W, const void* X, OutT* Y, int M, int N, i
 // first call; a non-zero value afterwards says a barrier wait ran out (1 copy, 2 MMA, 3 epilogue)
 // and the output is not valid.
 // `pair` = 1 uses pairs of blocks (256 x 256 tiles), 0 single blocks (128 x 256 tiles).
-// With out_kind 2, (limit, slope, shift) choose the gated activation (`GluParams`; limit 0: SwiGLU).
+// With out_kind 2, (limit, slope, shift, bias) choose the gated activation (`GluParams`; limit 0: SwiGLU; bias may be null).
 X0NE_API int x0ne_gemm_bf16_tcgen05_glu(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,
-                                        int pair, int* status, float limit, float slope, float shift, cudaStream_t stream) {
-    const GluParams glu = {limit, slope, shift};
+                                        int pair, int* status, float limit, float slope, float shift, const float* bias, cudaStream_t stream) {
+    const GluParams glu = {limit, slope, shift, bias};
     X0NE_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tc: M %d N %d K %d", M, N, K);
     X0NE_REQUIRE(K % 8 == 0, "gemm_tc: K %d is not a multiple of 8 (rows must be 16-byte aligned)", K);
     X0NE_REQUIRE(ldy >= N && out_kind >= 0 && out_kind <= 2 && status != nullptr, "gemm_tc: ldy %d N %d kind %d", ldy, N, out_kind);
@@ -522,5 +522,5 @@ X0NE_API int x0ne_gemm_bf16_tcgen05_glu(const void* W, const void* X, void* Y, i
 
 X0NE_API int x0ne_gemm_bf16_tcgen05(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,
                                     int pair, int* status, cudaStream_t stream) {
-    return x0ne_gemm_bf16_tcgen05_glu(W, X, Y, M, N, K, ldy, out_kind, pair, status, 0.f, 0.f, 0.f, stream);
+    return x0ne_gemm_bf16_tcgen05_glu(W, X, Y, M, N, K, ldy, out_kind, pair, status, 0.f, 0.f, 0.f, nullptr, stream);
 }

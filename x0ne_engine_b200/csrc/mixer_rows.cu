@@ -930,3 +930,159 @@ X0NE_API int x0ne_diff_heads(const float* att, const void* gate, int64_t gate_ld
         X0NE_REQUIRE(false, "diff_heads: unknown dtype tag %d", dt);
     X0NE_LAUNCH_CHECK();
 }
+
+// ----------------------------------------------------------------------------------------
+// Per-head preparation of an attention from a float32 projection: optional norm with a weight, rotate-half rotation of the
+// first `rot` values, values as they are.  src holds, per row of `ld` values, the queries at q_col (q_heads x dim), the keys
+// at k_col (kv_heads x dim) and the values at v_col (kv_heads x value width).
+//   n = x / sqrt(mean(x^2) + eps) * weight[d]   (weight null: n = x);  i < rot / 2, angle = pos * freq[i]:
+//   out[i] = n[i] cos - n[i + rot/2] sin;  out[i + rot/2] = n[i + rot/2] cos + n[i] sin;  the rest passes
+// Queries go to q_out [rows][q_heads][dim], keys and values into the pages, in the activation type, rounded once.  `table`
+// (float32 [positions][rot]: rot/2 cosines, then rot/2 sines) replaces the computation for the positions it covers.  One warp
+// per (row, query, key or value head); rows without a page write no keys or values.
+// ----------------------------------------------------------------------------------------
+struct HeadRopeArgs {
+    const float* src;
+    int64_t ld;
+    int32_t q_col, k_col, v_col;
+    const float* norm_q;
+    const float* norm_k;
+    float eps;
+    const float* freq;
+    const float* table;
+    int32_t table_positions, rot, q_heads, dim;
+    const int32_t* row_slot;
+    const int32_t* row_pos;
+    int32_t n_rows;
+};
+
+template <typename T, bool VEC>
+__global__ void head_norm_rope_kv_write_kernel(HeadRopeArgs a, T* __restrict__ q_out, PagedCache cache) {
+    extern __shared__ float hr_cs[];            // [warps][rot]: cosines, then sines (only without a table)
+    pdl_prologue();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int heads = a.q_heads + 2 * cache.kv_heads;
+    const int64_t item = (int64_t)blockIdx.x * (blockDim.x >> 5) + warp;
+    if (item >= (int64_t)a.n_rows * heads) return;
+    const int row = (int)(item / heads), head = (int)(item - (int64_t)row * heads);
+    const int pos = a.row_pos[row];
+    const float* src = a.src + (int64_t)row * a.ld;
+    if (head >= a.q_heads + cache.kv_heads) {           // a value head
+        const int kh = head - a.q_heads - cache.kv_heads, vd = cache_v_dim(cache);
+        const int64_t off = cache_row_offset(cache, a.row_slot[row], pos, kh, 1);
+        if (off < 0) return;
+        T* dst = (T*)cache.base + off;
+        src += a.v_col + (int64_t)kh * vd;
+        if (VEC) {
+            for (int i = 4 * lane; i < vd; i += 128) {
+                const float4 v = *reinterpret_cast<const float4*>(src + i);
+                const float y[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                for (int e = 0; e < 4; e += 2) {
+                    if (sizeof(T) == 2) *reinterpret_cast<__nv_bfloat162*>(dst + i + e) = __floats2bfloat162_rn(y[e], y[e + 1]);
+                    else *reinterpret_cast<float2*>(dst + i + e) = make_float2(y[e], y[e + 1]);
+                }
+            }
+        } else {
+            for (int i = lane; i < vd; i += 32) dst[i] = from_f32<T>(src[i]);
+        }
+        return;
+    }
+    const bool is_q = head < a.q_heads;
+    const int kh = head - a.q_heads, hd = a.dim, half = a.rot >> 1;
+    T* dst;
+    if (is_q) {
+        dst = q_out + ((int64_t)row * a.q_heads + head) * hd;
+        src += a.q_col + (int64_t)head * hd;
+    } else {
+        const int64_t off = cache_row_offset(cache, a.row_slot[row], pos, kh, 0);
+        if (off < 0) return;
+        dst = (T*)cache.base + off;
+        src += a.k_col + (int64_t)kh * hd;
+    }
+    const float* nw = is_q ? a.norm_q : a.norm_k;
+    const float* cs = nullptr;
+    if (a.rot > 0) {
+        if (a.table != nullptr && pos >= 0 && pos < a.table_positions) {
+            cs = a.table + (int64_t)pos * a.rot;
+        } else {
+            float* c = hr_cs + warp * a.rot;
+            for (int i = lane; i < half; i += 32) sincosf((float)pos * a.freq[i], &c[half + i], &c[i]);
+            __syncwarp();
+            cs = c;
+        }
+    }
+    float scale = 1.f;
+    if (nw != nullptr) {
+        float ss = 0.f;
+        for (int i = lane; i < hd; i += 32) ss = fmaf(src[i], src[i], ss);
+        scale = 1.0f / sqrtf(warp_sum(ss) / (float)hd + a.eps);
+    }
+    if (VEC) {
+        // pieces of 4 values; a rotated piece reads its partner half a turn on or back
+        for (int i = 4 * lane; i < hd; i += 128) {
+            const float4 x4 = *reinterpret_cast<const float4*>(src + i);
+            float x[4] = {x4.x, x4.y, x4.z, x4.w};
+            if (nw != nullptr) {
+                const float4 w4 = *reinterpret_cast<const float4*>(nw + i);
+                x[0] = x[0] * scale * w4.x; x[1] = x[1] * scale * w4.y; x[2] = x[2] * scale * w4.z; x[3] = x[3] * scale * w4.w;
+            }
+            if (i < a.rot) {
+                const bool first = i < half;
+                const int j = first ? i + half : i - half, at = first ? i : i - half;
+                const float4 y4 = *reinterpret_cast<const float4*>(src + j);
+                float y[4] = {y4.x, y4.y, y4.z, y4.w};
+                if (nw != nullptr) {
+                    const float4 w4 = *reinterpret_cast<const float4*>(nw + j);
+                    y[0] = y[0] * scale * w4.x; y[1] = y[1] * scale * w4.y; y[2] = y[2] * scale * w4.z; y[3] = y[3] * scale * w4.w;
+                }
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float c = cs[at + e], s = cs[half + at + e];
+                    x[e] = first ? x[e] * c - y[e] * s : x[e] * c + y[e] * s;
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+                if (sizeof(T) == 2) *reinterpret_cast<__nv_bfloat162*>(dst + i + e) = __floats2bfloat162_rn(x[e], x[e + 1]);
+                else *reinterpret_cast<float2*>(dst + i + e) = make_float2(x[e], x[e + 1]);
+            }
+        }
+    } else {
+    for (int i = lane; i < hd; i += 32) {
+        float x = src[i];
+        if (nw != nullptr) x = x * scale * nw[i];
+        if (i < a.rot) {
+            const bool first = i < half;
+            const int j = first ? i + half : i - half, at = first ? i : i - half;
+            float y = src[j];
+            if (nw != nullptr) y = y * scale * nw[j];
+            const float c = cs[at], s = cs[half + at];
+            x = first ? x * c - y * s : x * c + y * s;
+        }
+        dst[i] = from_f32<T>(x);
+    }
+    }
+}
+
+X0NE_API int x0ne_head_norm_rope_kv_write(HeadRopeArgs a, void* q_out, int dt, PagedCache cache, cudaStream_t stream) {
+    X0NE_REQUIRE(a.n_rows >= 0 && a.q_heads > 0 && a.dim > 0 && cache.kv_heads > 0 && cache.head_dim == a.dim && cache_v_dim(cache) > 0,
+                 "head_norm_rope: %d query heads of %d over a cache of %d heads of %d", a.q_heads, a.dim, cache.kv_heads, cache.head_dim);
+    X0NE_REQUIRE(a.rot >= 0 && a.rot % 2 == 0 && a.rot <= a.dim && (a.rot == 0 || a.freq != nullptr), "head_norm_rope: %d rotated values of %d", a.rot, a.dim);
+    X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "head_norm_rope: unknown dtype tag %d", dt);
+    if (a.n_rows == 0) return 0;
+    const int64_t items = (int64_t)a.n_rows * (a.q_heads + 2 * cache.kv_heads);
+    const dim3 grid((unsigned)((items + 3) / 4)), block(128);
+    const size_t smem = (size_t)4 * a.rot * sizeof(float);
+    const bool vec = a.dim % 4 == 0 && (a.rot / 2) % 4 == 0 && cache_v_dim(cache) % 4 == 0 && a.ld % 4 == 0 && a.q_col % 4 == 0 && a.k_col % 4 == 0 &&
+                     a.v_col % 4 == 0 && cache.page_stride % 4 == 0 &&
+                     (((uintptr_t)a.src | (uintptr_t)a.norm_q | (uintptr_t)a.norm_k | (uintptr_t)q_out | (uintptr_t)cache.base) & 15) == 0;
+    if (dt == X0NE_F32) {
+        if (vec) x0ne_launch(head_norm_rope_kv_write_kernel<float, true>, grid, block, smem, stream, a, (float*)q_out, cache);
+        else x0ne_launch(head_norm_rope_kv_write_kernel<float, false>, grid, block, smem, stream, a, (float*)q_out, cache);
+    } else {
+        if (vec) x0ne_launch(head_norm_rope_kv_write_kernel<bf16, true>, grid, block, smem, stream, a, (bf16*)q_out, cache);
+        else x0ne_launch(head_norm_rope_kv_write_kernel<bf16, false>, grid, block, smem, stream, a, (bf16*)q_out, cache);
+    }
+    X0NE_LAUNCH_CHECK();
+}

@@ -47,23 +47,39 @@ class AttnExtraArg(Structure):
     """Mirror of `struct AttnExtra` in common.cuh: what an attention kernel is asked for beyond causal
     softmax over a window (all zero: nothing)."""
     _fields_ = [("chunk", c_int32), ("v_from_k", c_int32), ("sink", c_void_p), ("gate", c_void_p),
-                ("gate_ld", c_int64), ("q_ld", c_int64), ("keep_first", c_int32), ("gate_wide", c_int32), ("slope", c_void_p), ("out_f32", c_int32)]
+                ("gate_ld", c_int64), ("q_ld", c_int64), ("keep_first", c_int32), ("gate_wide", c_int32), ("slope", c_void_p), ("out_f32", c_int32),
+                ("sig_bias", c_void_p), ("out_ld", c_int64), ("out_scale", c_float), ("out_col", c_int32)]
+
+    def out_width(self, heads_width: int) -> int:
+        """Values of a result row whose heads take `heads_width` of them; raises where they do not fit."""
+        width = int(self.out_ld) or heads_width
+        if self.out_col < 0 or self.out_col + heads_width > width:
+            raise KernelError("attention: the heads do not fit into the result rows")
+        return width
 
 
 def attn_extra(chunk: int = 0, v_from_k: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                gate_ld: int = 0, q_ld: int = 0, keep_first: int = 0, gate_wide: bool = False,
-               slope: Optional[torch.Tensor] = None, out_f32: bool = False) -> AttnExtraArg:
+               slope: Optional[torch.Tensor] = None, out_f32: bool = False, sig_bias: Optional[torch.Tensor] = None, out_ld: int = 0,
+               out_scale: float = 0.0, out_col: int = 0) -> AttnExtraArg:
     """`sink`: float32 per q head.  `gate`: a view whose element (row, head) lies at row * gate_ld + head; with
     `gate_wide` it holds a value per (row, head, value) at row * gate_ld + head * value width + value.
     `keep_first`: the keys at positions below it stay visible to every later query, whatever the window or chunk.
     `slope`: float32 per q head; slope[h] * (i - j) is taken off the scaled score of query i and key j.
-    `out_f32`: the results are written as float32 (the output tensor is float32) whatever the queries' type."""
+    `out_f32`: the results are written as float32 (the output tensor is float32) whatever the queries' type.
+    `sig_bias`: float32 per q head; instead of the softmax key j weighs sigmoid(score + sig_bias[h]) and nothing is normalised
+    over the keys.  `out_ld`: values between result rows that are wider than the heads, which start at `out_col`.
+    `out_scale`: the results are multiplied by it (0: by one)."""
+    if sig_bias is not None:
+        _need(sig_bias, torch.float32, "score biases")
+        if sink is not None:
+            raise KernelError("attention: weights that nothing normalises have no denominator for a sink to join")
     if sink is not None:
         _need(sink, torch.float32, "sink")
     if slope is not None:
         _need(slope, torch.float32, "distance slopes")
     return AttnExtraArg(int(chunk or 0), int(v_from_k or 0), _ptr(sink), _ptr(gate), int(gate_ld), int(q_ld), int(keep_first or 0),
-                        1 if gate_wide else 0, _ptr(slope), 1 if out_f32 else 0)
+                        1 if gate_wide else 0, _ptr(slope), 1 if out_f32 else 0, _ptr(sig_bias), int(out_ld), float(out_scale), int(out_col))
 
 
 class SsmArg(Structure):
@@ -72,6 +88,49 @@ class SsmArg(Structure):
                 ("A", c_void_p), ("bc", c_void_p), ("bc_ld", c_int64), ("b_col", c_int32), ("c_col", c_int32), ("D", c_void_p),
                 ("out", c_void_p), ("state", c_void_p), ("state_stride", c_int64), ("conv_off", c_int64), ("seq_first_row", c_void_p),
                 ("seq_slot", c_void_p), ("channels", c_int32), ("N", c_int32), ("taps", c_int32)]
+
+
+class GatedScanArg(Structure):
+    """Mirror of `struct GatedScanArgs` in gated_scan.cu."""
+    _fields_ = [("q", c_void_p), ("k", c_void_p), ("w", c_void_p), ("v", c_void_p), ("q_ld", c_int64), ("k_ld", c_int64), ("w_ld", c_int64),
+                ("v_ld", c_int64), ("gates", c_void_p), ("o", c_void_p), ("nq", c_void_p), ("state", c_void_p), ("state_stride", c_int64),
+                ("seq_first_row", c_void_p), ("seq_slot", c_void_p), ("heads", c_int32), ("D", c_int32), ("V", c_int32), ("C", c_int32)]
+
+
+class GatedRawArg(Structure):
+    """Mirror of `struct GatedRaw` in gated_scan.cu."""
+    _fields_ = [("src", c_void_p), ("ld", c_int64), ("q_col", c_int32), ("k_col", c_int32), ("v_col", c_int32), ("i_col", c_int32),
+                ("f_col", c_int32), ("f_bias", c_void_p), ("i_bias", c_void_p), ("lower", c_void_p), ("cap", c_float), ("m_off", c_int64),
+                ("em", c_void_p), ("seq_pos0", c_void_p)]
+
+
+class HeadNormArg(Structure):
+    """Mirror of `struct HeadNormArgs` in gated_scan.cu."""
+    _fields_ = [("o", c_void_p), ("nq", c_void_p), ("em", c_void_p), ("q_scale", c_float), ("tiny", c_float), ("weight", c_void_p),
+                ("shared", c_int32), ("gate", c_void_p), ("gate_ld", c_int64), ("eps", c_float), ("post", c_float), ("out_ld", c_int64),
+                ("heads", c_int32), ("V", c_int32)]
+
+
+class HeadRopeArg(Structure):
+    """Mirror of `struct HeadRopeArgs` in mixer_rows.cu."""
+    _fields_ = [("src", c_void_p), ("ld", c_int64), ("q_col", c_int32), ("k_col", c_int32), ("v_col", c_int32), ("norm_q", c_void_p),
+                ("norm_k", c_void_p), ("eps", c_float), ("freq", c_void_p), ("table", c_void_p), ("table_positions", c_int32),
+                ("rot", c_int32), ("q_heads", c_int32), ("dim", c_int32), ("row_slot", c_void_p), ("row_pos", c_void_p), ("n_rows", c_int32)]
+
+
+class EmbedSumArg(Structure):
+    """Mirror of `struct EmbedSumArgs` in elementwise.cu."""
+    _fields_ = [("table", c_void_p), ("pairs", c_void_p), ("positions", c_void_p), ("tokens", c_void_p), ("row_slot", c_void_p),
+                ("row_pos", c_void_p), ("seq_first_row", c_void_p), ("last_token", c_void_p), ("state_stride", c_int64), ("resid", c_void_p),
+                ("copy", c_void_p), ("mul_prev", c_int64), ("mul_cur", c_int64), ("buckets", c_int64), ("n_seqs", c_int32), ("hidden", c_int32),
+                ("vocab", c_int32), ("n_positions", c_int32)]
+
+
+class NormConvArg(Structure):
+    """Mirror of `struct NormConvArgs` in input_conv.cu."""
+    _fields_ = [("resid", c_void_p), ("delta", c_void_p), ("bias_d", c_void_p), ("w_d", c_void_p), ("eps_d", c_float), ("w", c_void_p),
+                ("eps", c_float), ("conv", c_void_p), ("state", c_void_p), ("state_stride", c_int64), ("off", c_int64), ("row_slot", c_void_p),
+                ("width", c_int32), ("taps", c_int32)]
 
 
 class SampleIOArg(Structure):
@@ -91,7 +150,18 @@ _P, _I, _F, _L = c_void_p, c_int, c_float, c_int64
 # and per call (1.4 us against 3.8 us for ten arguments).  Pointers are passed as integers.
 _SIGNATURES = {
     "x0ne_embedding": [_P, _I, _P, _P, _I, _I, _I, _F, _P],
-    "x0ne_add_normed_rmsnorm": [_P, _P, _P, _F, _P, _P, _I, _P, _I, _I, _F, _P],
+    "x0ne_gated_scan": [GatedScanArg, _I, _P],
+    "x0ne_gated_step": [GatedScanArg, GatedRawArg, _I, _P],
+    "x0ne_channel_gates": [GatedRawArg, _P, _I, _I, _P],
+    "x0ne_head_gates": [GatedRawArg, _P, _P, _L, _P, _P, _I, _I, _P],
+    "x0ne_scan_head_norm": [HeadNormArg, _P, _I, _I, _P],
+    "x0ne_head_norm_rope_kv_write": [HeadRopeArg, _P, _I, None, _P],
+    "x0ne_embed_sum": [EmbedSumArg, _I, _I, _P],
+    "x0ne_concat_rows": [_P, _P, _I, _P, _P, _F, _P, _P, _I, _I, _I, _P],
+    "x0ne_add_f32": [_P, _P, _P, _L, _P],
+    "x0ne_input_conv": [_P, _I, _P, _P, _L, _L, _P, _P, _P, _I, _I, _I, _I, _P],
+    "x0ne_norm_conv_step": [NormConvArg, _P, _I, _I, _P],
+    "x0ne_add_normed_rmsnorm": [_P, _P, _P, _P, _F, _P, _P, _I, _P, _I, _I, _F, _P],
     "x0ne_whole_norm_rope_kv_write": [_P, _I, _I, _I, _I, _P, _P, _F, _P, _I, _P, _I, _P, _I, None, _P, _P, _I, _I, _P],
     "x0ne_relu2": [_P, _P, _I, _L, _P],
     "x0ne_moe_route": [_P, _I, _P, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P],
@@ -122,16 +192,16 @@ _SIGNATURES = {
     "x0ne_attention_flex_prefill": [_P, _P, None, _P, _P, _I, _P, _P, _P, _I, _F, _I, "ex", _P],
     "x0ne_attention_flex_decode": [_P, _P, None, _P, _P, _I, _I, _F, _I, "ex", _I, _P, _L, _P],
     "x0ne_qk_norm_rope_kv_write": [_P, _I, _P, _P, _P, _I, _P, None, _P, _P, _I, _I, _F, _I, _P, _I, _P],
-    "x0ne_swiglu": [_P, _P, _I, _I, _I, _P],
+    "x0ne_swiglu": [_P, _P, _P, _I, _I, _I, _P],
     "x0ne_attention_rows": [_P, _P, _I, None, _P, _P, _I, _I, _F, _I, _P],
     "x0ne_gemm_f32_nt": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "x0ne_attention_prefill_bf16": [_P, _P, None, _P, _P, _I, _P, _P, _P, _I, _F, _I, _P],
     "x0ne_attention_decode_bf16": [_P, _P, None, _P, _P, _I, _I, _F, _I, _I, _P, _L, _P],
     "x0ne_attention_decode_grouped_bf16": [_P, _P, None, _P, _P, _I, _I, _F, _I, _I, _I, _P, _L, _P],
     "x0ne_gemm_bf16_smallm": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-    "x0ne_gemm_bf16_smallm_glu": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
-    "x0ne_gemm_bf16_tcgen05_glu": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _F, _F, _F, _P],
-    "x0ne_gemm_bf16_skinny_tcgen05_glu": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _P, _F, _F, _F, _P],
+    "x0ne_gemm_bf16_smallm_glu": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
+    "x0ne_gemm_bf16_tcgen05_glu": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _F, _F, _F, _P, _P],
+    "x0ne_gemm_bf16_skinny_tcgen05_glu": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _P, _F, _F, _F, _P, _P],
     "x0ne_attention_prefill_tcgen05": [_P, _P, _I, None, _P, _P, _I, _P, _P, _P, _I, _F, _I, _P, _P],
     "x0ne_gemm_bf16_tcgen05": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     "x0ne_gemm_bf16_skinny_tcgen05": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _P, _P],
@@ -274,8 +344,8 @@ def add_rmsnorm(resid: torch.Tensor, delta, weight: torch.Tensor, out: torch.Ten
 
 def add_normed_rmsnorm(resid: torch.Tensor, delta: torch.Tensor, delta_weight: torch.Tensor, delta_eps: float,
                        weight: torch.Tensor, out: torch.Tensor, n_rows: int, eps: float,
-                       rows: Optional[torch.Tensor] = None) -> None:
-    """resid += rmsnorm(delta) * delta_weight (float32, never rounded); out = rmsnorm(resid) * weight.  `rows`
+                       rows: Optional[torch.Tensor] = None, delta_bias: Optional[torch.Tensor] = None) -> None:
+    """resid += rmsnorm(delta + delta_bias) * delta_weight (float32, never rounded); out = rmsnorm(resid) * weight.  `rows`
     gathers source rows."""
     lib = _lib("core")
     hidden = weight.numel()
@@ -293,7 +363,11 @@ def add_normed_rmsnorm(resid: torch.Tensor, delta: torch.Tensor, delta_weight: t
             raise KernelError("add_normed_rmsnorm: row list shorter than the rows asked for")
     elif resid.numel() < n_rows * hidden or delta.numel() < n_rows * hidden:
         raise KernelError("add_normed_rmsnorm: residual or delta smaller than the rows asked for")
-    _check(lib, lib.x0ne_add_normed_rmsnorm(_ptr(resid), _ptr(delta), _ptr(delta_weight), delta_eps, _ptr(weight), _ptr(out),
+    if delta_bias is not None:
+        _need(delta_bias, torch.float32, "delta bias")
+        if delta_bias.numel() != hidden:
+            raise KernelError("add_normed_rmsnorm: the delta's bias does not have its width")
+    _check(lib, lib.x0ne_add_normed_rmsnorm(_ptr(resid), _ptr(delta), _ptr(delta_bias), _ptr(delta_weight), delta_eps, _ptr(weight), _ptr(out),
                                             dtype_tag(out.dtype), _ptr(rows), n_rows, hidden, eps, _stream()),
            "add_normed_rmsnorm")
 
@@ -534,7 +608,8 @@ def attention_rows(q: torch.Tensor, out: torch.Tensor, cache: PagedCacheArg, row
     if not q.is_cuda or (extra is None or not extra.q_ld) and not q.is_contiguous():
         raise KernelError("attention: q is not a contiguous GPU tensor")
     vd = extra.v_from_k if extra is not None and extra.v_from_k else cache.value_dim
-    width, out_width = q_heads * cache.head_dim, q_heads * vd
+    width = q_heads * cache.head_dim
+    out_width = q_heads * vd if extra is None else extra.out_width(q_heads * vd)
     if extra is None or not extra.q_ld:
         if q.shape[-1] != width or q.numel() < n_rows * width:
             raise KernelError("attention: q does not match the head counts and rows")
@@ -690,7 +765,7 @@ def attention_flex_prefill(q: torch.Tensor, out: torch.Tensor, cache: PagedCache
     if tile_seq.numel() < n_tiles or tile_row0.numel() < n_tiles:
         raise KernelError("attention_flex: tile tables shorter than the tiles asked for")
     vd = extra.v_from_k or cache.value_dim
-    if out.shape[-1] != q_heads * vd:
+    if out.shape[-1] != extra.out_width(q_heads * vd):
         raise KernelError("attention_flex: the output width does not match the head counts")
     for first in range(0, n_tiles, 65535):
         n = min(65535, n_tiles - first)
@@ -716,7 +791,7 @@ def attention_flex_decode(q: torch.Tensor, out: torch.Tensor, cache: PagedCacheA
     _need(row_slot, torch.int32, "row slots")
     _need(row_pos, torch.int32, "row positions")
     vd = extra.v_from_k or cache.value_dim
-    if out.shape[-1] != q_heads * vd or out.numel() < n_rows * q_heads * vd or row_slot.numel() < n_rows or row_pos.numel() < n_rows:
+    if out.shape[-1] != extra.out_width(q_heads * vd) or out.numel() < n_rows * out.shape[-1] or row_slot.numel() < n_rows or row_pos.numel() < n_rows:
         raise KernelError("attention_flex: output or row tables do not match the rows asked for")
     nbytes = scratch.numel() * scratch.element_size() if scratch is not None else 0
     _check(lib, lib.x0ne_attention_flex_decode(_ptr(q), _ptr(out), cache, _ptr(row_slot), _ptr(row_pos), n_rows, q_heads,
@@ -727,14 +802,23 @@ def attention_flex_decode(q: torch.Tensor, out: torch.Tensor, cache: PagedCacheA
         LAUNCHES += 1
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, n_rows: int) -> None:
+def _glu_bias(bias: Optional[torch.Tensor], n: int) -> None:
+    if bias is not None:
+        _need(bias, torch.float32, "biases of a gated unit")
+        if bias.numel() != 2 * n:
+            raise KernelError(f"a gated unit of {n} outputs needs {2 * n} biases (gate, then up), got {bias.numel()}")
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, n_rows: int, bias: Optional[torch.Tensor] = None) -> None:
+    """out = silu(gate + its bias) * (up + its bias) on packed [gate; up] rows; `bias` is packed alike (float32)."""
     lib = _lib("core")
+    _glu_bias(bias, out.shape[-1])
     _need(gate_up, gate_up.dtype, "gate_up")
     _need(out, gate_up.dtype, "swiglu output")
     inter = out.shape[-1]
     if gate_up.shape[-1] != 2 * inter or gate_up.numel() < n_rows * 2 * inter or out.numel() < n_rows * inter:
         raise KernelError("swiglu: widths or rows do not match")
-    _check(lib, lib.x0ne_swiglu(_ptr(gate_up), _ptr(out), dtype_tag(out.dtype), n_rows, inter,
+    _check(lib, lib.x0ne_swiglu(_ptr(gate_up), _ptr(bias), _ptr(out), dtype_tag(out.dtype), n_rows, inter,
                                 _stream()), "swiglu")
 
 
@@ -892,6 +976,16 @@ def attention_decode_bf16(q: torch.Tensor, out: torch.Tensor, cache: PagedCacheA
 # ---------------------------------------------------------------------------------------------
 # bfloat16 small-M weight-streaming product (module `fast`)
 # ---------------------------------------------------------------------------------------------
+def _glu_of(glu: Optional[tuple], bias: Optional[torch.Tensor], n: int, swiglu: bool) -> Optional[tuple]:
+    """(limit, slope, shift) of a product's gated epilogue that has biases (limit 0: SwiGLU), or `glu` as it is."""
+    if bias is None:
+        return glu
+    if not swiglu:
+        raise KernelError("biases belong to a gated epilogue")
+    _glu_bias(bias, n)
+    return glu if glu is not None else (0.0, 0.0, 0.0)
+
+
 SMALL_M_MAX_ROWS = 32       # rows the weight-streaming kernel takes (which products use it: routes.py)
 _sm_count = {}
 
@@ -910,7 +1004,7 @@ def gemm_smallm_takes(w: torch.Tensor, m: int, swiglu: bool = False) -> bool:
 
 
 def gemm_bf16_smallm(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, swiglu: bool = False,
-                     glu: Optional[tuple] = None) -> None:
+                     glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None) -> None:
     """y[:m] = x[:m] @ w.T for m <= 32 by streaming w once; y is bfloat16 or float32.  With
     `swiglu`, w is the packed [gate; up] weight and y[:m] = silu(x gate^T) * (x up^T); with `glu` =
     (limit, slope, shift) besides, the clipped unit min(g, limit) sigmoid(slope g) (clamp(u) + shift)."""
@@ -928,9 +1022,10 @@ def gemm_bf16_smallm(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, 
         kind = 2 if swiglu else 0
     else:
         raise KernelError(f"gemm_smallm: no output kind for {y.dtype} (swiglu={swiglu})")
+    glu = _glu_of(glu, bias, n, swiglu)
     if glu is not None and swiglu:
         _check(lib, lib.x0ne_gemm_bf16_smallm_glu(_ptr(w), _ptr(x), _ptr(y), m, n, k, n, kind, _sms(w.device),
-                                                  glu[0], glu[1], glu[2], _stream()), "gemm_bf16_smallm")
+                                                  glu[0], glu[1], glu[2], _ptr(bias), _stream()), "gemm_bf16_smallm")
         return
     _check(lib, lib.x0ne_gemm_bf16_smallm(_ptr(w), _ptr(x), _ptr(y), m, n, k, n,
                                           kind, _sms(w.device), _stream()), "gemm_bf16_smallm")
@@ -979,7 +1074,7 @@ def gemm_tc_status(device) -> torch.Tensor:
 
 
 def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, swiglu: bool = False,
-                      pair: bool = True, glu: Optional[tuple] = None) -> None:
+                      pair: bool = True, glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None) -> None:
     """y[:m] = x[:m] @ w.T on the tcgen05 tensor cores (128 x 256 tiles, TMA loads, accumulator in
     tensor memory; with `pair`, pairs of blocks on 256 x 256 tiles); y is bfloat16 or float32.  With `swiglu`, w is the packed [gate; up] weight and
     y[:m] = silu(x gate^T) * (x up^T).  Needs K % 8 == 0."""
@@ -999,9 +1094,10 @@ def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int,
         raise KernelError(f"gemm_tc: no output kind for {y.dtype} (swiglu={swiglu})")
     global tc_used
     tc_used = True
+    glu = _glu_of(glu, bias, n, swiglu)
     if glu is not None and swiglu:       # (limit, slope, shift): the clipped gated unit instead of SwiGLU
         _check(lib, lib.x0ne_gemm_bf16_tcgen05_glu(_ptr(w), _ptr(x), _ptr(y), m, n, k, n, kind, 1 if pair else 0,
-                                                   _ptr(gemm_tc_status(w.device)), glu[0], glu[1], glu[2], _stream()),
+                                                   _ptr(gemm_tc_status(w.device)), glu[0], glu[1], glu[2], _ptr(bias), _stream()),
                "gemm_bf16_tcgen05")
         return
     _check(lib, lib.x0ne_gemm_bf16_tcgen05(_ptr(w), _ptr(x), _ptr(y), m, n, k, n,
@@ -1029,7 +1125,7 @@ def product_kernel(w: torch.Tensor, m: int, fused: bool = False) -> str:
 
 
 def gemm_bf16_skinny_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, swiglu: bool = False,
-                             glu: Optional[tuple] = None) -> None:
+                             glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None) -> None:
     """y[:m] = x[:m] @ w.T for up to 64 rows on tcgen05, K cut over the blocks of a cluster that add
     their partial sums through shared memory; y is bfloat16 or float32.  With `swiglu`, w is the
     packed [gate; up] weight and y[:m] = silu(x gate^T) * (x up^T).  Failures of its bounded waits
@@ -1051,9 +1147,10 @@ def gemm_bf16_skinny_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, 
         raise KernelError(f"gemm_skinny_tc: no output kind for {y.dtype} (swiglu={swiglu})")
     tc_used = True
     x_rows = x.numel() // k      # rows really behind x: the copies may read them all (their results are not used)
+    glu = _glu_of(glu, bias, n, swiglu)
     if glu is not None and swiglu:       # (limit, slope, shift): the clipped gated unit instead of SwiGLU
         _check(lib, lib.x0ne_gemm_bf16_skinny_tcgen05_glu(_ptr(w), _ptr(x), x_rows, _ptr(y), m, n, k, n, kind,
-                                                          _ptr(gemm_tc_status(x.device)), glu[0], glu[1], glu[2], _stream()),
+                                                          _ptr(gemm_tc_status(x.device)), glu[0], glu[1], glu[2], _ptr(bias), _stream()),
                "gemm_bf16_skinny_tcgen05")
         return
     _check(lib, lib.x0ne_gemm_bf16_skinny_tcgen05(_ptr(w), _ptr(x), x_rows, _ptr(y), m, n, k, n, kind,
@@ -1315,3 +1412,257 @@ def selective_scan(u: torch.Tensor, xz: torch.Tensor, z_col: int, dt_raw: torch.
                  int(c_col), _ptr(D), _ptr(out), _ptr(state), state.stride(0), int(conv_off), _ptr(seq_first_row), _ptr(seq_slot),
                  int(channels), int(N), int(taps))
     _check(lib, lib.x0ne_selective_scan(arg, dtype_tag(u.dtype), n_seqs, 1 if one_token else 0, _stream()), "selective_scan")
+
+
+# ---------------------------------------------------------------------------------------------
+# embedding as a sum of rows, operand of a product over concatenated rows, input convolution (module `core`)
+# ---------------------------------------------------------------------------------------------
+def embed_sum(table: torch.Tensor, pairs: Optional[torch.Tensor], positions: Optional[torch.Tensor], tokens: torch.Tensor, resid: torch.Tensor,
+              copy: Optional[torch.Tensor], last_token: Optional[torch.Tensor], mul_prev: int, mul_cur: int, row_slot: torch.Tensor,
+              row_pos: torch.Tensor, seq_first_row: torch.Tensor, n_seqs: int, n_rows: int) -> None:
+    """resid[r] = table[token] + pairs[(previous token * mul_prev + token * mul_cur) mod buckets] + positions[pos], float32;
+    `pairs` has buckets + 1 rows, the last for a sequence's first token.  `last_token` (float32 [slots, 1], its bits an
+    int32) is what a sequence keeps of its previous token.  `copy` receives the rows too."""
+    lib = _lib("core")
+    _need(tokens, torch.int32, "tokens")
+    _need(resid, torch.float32, "residual")
+    vocab, hidden = table.shape
+    for t, what in ((table, "embedding table"), (pairs, "pair rows"), (positions, "position rows")):
+        if t is not None:
+            _need(t, table.dtype, what)
+            if t.dim() != 2 or t.shape[1] != hidden:
+                raise KernelError(f"embed_sum: the {what} do not have the residual's width")
+    if pairs is not None:
+        _need(last_token, torch.float32, "previous tokens")
+        if not (0 <= mul_prev < 1 << 31 and 0 <= mul_cur < 1 << 31):
+            raise KernelError("embed_sum: a multiplier lies outside 31 bits")
+    if copy is not None:
+        _need(copy, torch.float32, "copy of the rows")
+        if copy.numel() < n_rows * hidden:
+            raise KernelError("embed_sum: the copy is smaller than the rows asked for")
+    if resid.shape[-1] != hidden or resid.numel() < n_rows * hidden or tokens.numel() < n_rows:
+        raise KernelError("embed_sum: buffers are smaller than the rows asked for")
+    arg = EmbedSumArg(_ptr(table), _ptr(pairs), _ptr(positions), _ptr(tokens), _ptr(row_slot), _ptr(row_pos), _ptr(seq_first_row),
+                      _ptr(last_token) if pairs is not None else None, last_token.stride(0) if pairs is not None else 0, _ptr(resid), _ptr(copy),
+                      int(mul_prev), int(mul_cur), pairs.shape[0] - 1 if pairs is not None else 0, n_seqs, hidden, vocab,
+                      positions.shape[0] if positions is not None else 0)
+    _check(lib, lib.x0ne_embed_sum(arg, dtype_tag(table.dtype), n_rows, _stream()), "embed_sum")
+
+
+def concat_rows(resid: torch.Tensor, delta: Optional[torch.Tensor], delta_bias: Optional[torch.Tensor], delta_weight: Optional[torch.Tensor],
+                delta_eps: float, x0: torch.Tensor, out: torch.Tensor, n_rows: int, lo: bool = False) -> None:
+    """out[r] = [x | x0[r]] with x = resid[r] + rmsnorm(delta[r] + delta_bias) * delta_weight (no weight: delta is added as it
+    is; no delta: resid alone), rounded once to out's type; `lo`: rows n_rows .. 2 n_rows - 1 receive what that lost."""
+    lib = _lib("core")
+    _need(resid, torch.float32, "residual")
+    _need(x0, torch.float32, "second rows")
+    _need(out, out.dtype, "concatenated rows")
+    hidden = resid.shape[-1]
+    if delta is not None:
+        _need(delta, out.dtype, "delta")
+    for t, what in ((delta_bias, "delta bias"), (delta_weight, "norm weight of the delta")):
+        if t is not None:
+            _need(t, torch.float32, what)
+    if out.shape[-1] != 2 * hidden or out.numel() < (2 if lo else 1) * n_rows * 2 * hidden or x0.numel() < n_rows * hidden or resid.numel() < n_rows * hidden:
+        raise KernelError("concat_rows: shapes do not match")
+    _check(lib, lib.x0ne_concat_rows(_ptr(resid), _ptr(delta), dtype_tag(out.dtype), _ptr(delta_bias), _ptr(delta_weight), float(delta_eps),
+                                     _ptr(x0), _ptr(out), n_rows, hidden, 1 if lo else 0, _stream()), "concat_rows")
+
+
+def add_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, total: int) -> None:
+    """out[i] = a[i] + b[i] for the first `total` values."""
+    lib = _lib("core")
+    for t in (a, b, out):
+        _need(t, torch.float32, "float32 rows")
+        if t.numel() < total:
+            raise KernelError("add_f32: fewer values than asked for")
+    _check(lib, lib.x0ne_add_f32(_ptr(a), _ptr(b), _ptr(out), total, _stream()), "add_f32")
+
+
+INPUT_CONV_MAX_TAPS = 17
+
+
+def input_conv(h: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor], out: torch.Tensor, seq_first_row: torch.Tensor,
+               seq_slot: torch.Tensor, n_seqs: int, max_seq_rows: int) -> None:
+    """out[t] = h[t] + sum_j w[j] * h[t - (K - 1) + j] per channel over the rows of every sequence; w float32 [K, width]; inputs
+    ahead of the pass come from `state` (float32 [slots, (K - 1) * width], oldest first), which is brought up to date."""
+    lib = _lib("core")
+    _need(h, h.dtype, "convolution input")
+    _need(out, h.dtype, "convolution output")
+    _need(w, torch.float32, "convolution taps")
+    taps, width = w.shape
+    if state is not None:
+        _need(state, torch.float32, "convolution state")
+    if h.shape[-1] != width or out.shape[-1] != width or (taps > 1 and (state is None or state.dim() != 2 or state.shape[1] < (taps - 1) * width)):
+        raise KernelError("input_conv: shapes do not match")
+    _check(lib, lib.x0ne_input_conv(_ptr(h), dtype_tag(h.dtype), _ptr(w), _ptr(state), state.stride(0) if state is not None else 0, 0, _ptr(out),
+                                    _ptr(seq_first_row), _ptr(seq_slot), n_seqs, max_seq_rows, width, taps, _stream()), "input_conv")
+
+
+def norm_conv_step_takes(width: int) -> bool:
+    return width % 8 == 0 and width <= 8 * 1024 * 2
+
+
+def norm_conv_step(resid: torch.Tensor, delta: Optional[torch.Tensor], delta_bias: Optional[torch.Tensor], delta_weight: Optional[torch.Tensor],
+                   delta_eps: float, weight: torch.Tensor, eps: float, conv: torch.Tensor, state: Optional[torch.Tensor], out: torch.Tensor,
+                   row_slot: torch.Tensor, n_rows: int) -> None:
+    """One row per sequence: resid += rmsnorm(delta + delta_bias) * delta_weight (no delta: nothing is added); h =
+    rmsnorm(resid) * weight; out = h + convolution of h with the inputs `state` keeps, which h joins (see input_conv)."""
+    lib = _lib("core")
+    _need(resid, torch.float32, "residual")
+    _need(out, out.dtype, "convolution output")
+    for t, what in ((weight, "norm weight"), (conv, "convolution taps")):
+        _need(t, torch.float32, what)
+    for t, what in ((delta_bias, "delta bias"), (delta_weight, "norm weight of the delta"), (state, "convolution state")):
+        if t is not None:
+            _need(t, torch.float32, what)
+    if delta is not None:
+        _need(delta, out.dtype, "delta")
+    taps, width = conv.shape
+    if resid.shape[-1] != width or out.shape[-1] != width or weight.numel() != width or resid.numel() < n_rows * width \
+            or (taps > 1 and (state is None or state.shape[1] < (taps - 1) * width)):
+        raise KernelError("norm_conv_step: shapes do not match")
+    arg = NormConvArg(_ptr(resid), _ptr(delta), _ptr(delta_bias), _ptr(delta_weight), float(delta_eps), _ptr(weight), float(eps), _ptr(conv),
+                      _ptr(state), state.stride(0) if state is not None else 0, 0, _ptr(row_slot), width, taps)
+    _check(lib, lib.x0ne_norm_conv_step(arg, _ptr(out), dtype_tag(out.dtype), n_rows, _stream()), "norm_conv_step")
+
+
+def head_norm_rope_kv_write(src: torch.Tensor, q_col: int, k_col: int, v_col: int, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor],
+                            eps: float, freq: Optional[torch.Tensor], table: Optional[torch.Tensor], rot: int, q_out: torch.Tensor, q_heads: int,
+                            cache: PagedCacheArg, row_slot: torch.Tensor, row_pos: torch.Tensor, n_rows: int) -> None:
+    """Queries, keys and values of the float32 projection `src` (columns from q_col, k_col, v_col): each query and key head over
+    its root mean square times q_norm / k_norm (None: as it is), the first `rot` values of every head turned as pairs (i,
+    i + rot / 2) by pos * freq[i] (`table`: float32 [positions, rot], cosines then sines), values as they are; queries to q_out,
+    keys and values to the pages, in q_out's type."""
+    lib = _lib("core")
+    _need(src, torch.float32, "projection")
+    _need(q_out, q_out.dtype, "queries")
+    dim = cache.head_dim
+    for t, what in ((q_norm, "query norm"), (k_norm, "key norm")):
+        if t is not None:
+            _need(t, torch.float32, what)
+            if t.numel() != dim:
+                raise KernelError("head_norm_rope_kv_write: a norm weight does not have a head's width")
+    if rot and (freq is None or freq.numel() < rot // 2):
+        raise KernelError("head_norm_rope_kv_write: fewer frequencies than pairs")
+    if freq is not None:
+        _need(freq, torch.float32, "rotary frequencies")
+    if table is not None:
+        _need(table, torch.float32, "rotary table")
+        if table.dim() != 2 or table.shape[1] != rot:
+            raise KernelError("head_norm_rope_kv_write: the table's rows do not hold rot values")
+    ends = (q_col + q_heads * dim, k_col + cache.kv_heads * dim, v_col + cache.kv_heads * cache.value_dim)
+    if max(ends) > src.shape[-1] or src.numel() < n_rows * src.shape[-1] or q_out.shape[-1] != q_heads * dim or q_out.numel() < n_rows * q_heads * dim:
+        raise KernelError("head_norm_rope_kv_write: buffers smaller than the rows asked for")
+    arg = HeadRopeArg(_ptr(src), src.shape[-1], q_col, k_col, v_col, _ptr(q_norm), _ptr(k_norm), float(eps), _ptr(freq), _ptr(table),
+                      0 if table is None else table.shape[0], rot, q_heads, dim, _ptr(row_slot), _ptr(row_pos), n_rows)
+    _check(lib, lib.x0ne_head_norm_rope_kv_write(arg, _ptr(q_out), dtype_tag(q_out.dtype), cache, _stream()), "head_norm_rope_kv_write")
+
+
+# ---------------------------------------------------------------------------------------------
+# gated linear attention with a matrix state per head (csrc/gated_scan.cu, module `core`)
+# ---------------------------------------------------------------------------------------------
+GATED_STEP_MAX_DIM = 256
+
+
+class GatedState:
+    """Where a gated scan's parts lie: the widths of a head, and for gates per head the place of the running maxima."""
+
+    def __init__(self, heads: int, dim: int, v_dim: int, head_gates: bool):
+        self.heads, self.dim, self.v_dim, self.head_gates = heads, dim, v_dim, head_gates
+        self.cols = v_dim + (1 if head_gates else 0)
+        self.m_off = heads * self.cols * dim
+        self.floats = -(-(self.m_off + (2 * heads if head_gates else 0)) // 4) * 4       # (rows of 16 bytes)
+
+    def heads_of(self, state_row: torch.Tensor) -> torch.Tensor:
+        """[..., heads, columns, dim] of state rows: the transposed state, the key sum as its last column."""
+        return state_row[..., :self.m_off].reshape(*state_row.shape[:-1], self.heads, self.cols, self.dim)
+
+
+def gated_raw(src: torch.Tensor, q_col: int, k_col: int, v_col: int, f_bias: torch.Tensor, lower: Optional[torch.Tensor] = None, i_col: int = 0,
+              f_col: int = 0, i_bias: Optional[torch.Tensor] = None, cap: float = 0.0, geometry: Optional[GatedState] = None,
+              em: Optional[torch.Tensor] = None, seq_pos0: Optional[torch.Tensor] = None) -> GatedRawArg:
+    """The raw inputs of a gated scan in the float32 projection `src`.  Gates per channel: k_col is the forget gates' column,
+    `lower` and f_bias hold a value per channel.  Gates per head: i_col, f_col, i_bias, f_bias, cap; `em` receives exp(-m)."""
+    for t, what in ((src, "projection"), (f_bias, "forget gate bias"), (lower, "lower bounds"), (i_bias, "input gate bias"), (em, "maxima")):
+        if t is not None:
+            _need(t, torch.float32, what)
+    return GatedRawArg(_ptr(src), src.shape[-1], q_col, k_col, v_col, i_col, f_col, _ptr(f_bias), _ptr(i_bias), _ptr(lower), float(cap),
+                       0 if geometry is None else geometry.m_off, _ptr(em), _ptr(seq_pos0))
+
+
+def _gated_arg(g: GatedState, o, nq, state, seq_first_row, seq_slot) -> GatedScanArg:
+    for t, what in ((o, "scan output"), (state, "state"), (nq, "key sums")):
+        if t is not None:
+            _need(t, torch.float32, what)
+    if state.dim() != 2 or state.shape[1] < g.floats or o.shape[-1] != g.heads * g.v_dim or (g.head_gates and (nq is None or nq.shape[-1] != g.heads)):
+        raise KernelError("gated scan: the state or an output does not have the heads' sizes")
+    return GatedScanArg(None, None, None, None, 0, 0, 0, 0, None, _ptr(o), _ptr(nq), _ptr(state), state.stride(0), _ptr(seq_first_row), _ptr(seq_slot),
+                        g.heads, g.dim, g.v_dim, g.cols)
+
+
+def gated_scan(g: GatedState, q: torch.Tensor, k: torch.Tensor, w: Optional[torch.Tensor], v: torch.Tensor, gates: Optional[torch.Tensor],
+               o: torch.Tensor, nq: Optional[torch.Tensor], state: torch.Tensor, seq_first_row: torch.Tensor, seq_slot: torch.Tensor,
+               n_seqs: int) -> None:
+    """Token by token over every sequence's rows, from and into its state:  S = w S + k v^T, o = S^T q per head.  q, k, w
+    (per channel, or None) and v are float32 views whose row r starts stride(0) values after row r - 1 and whose first value is
+    head 0's; `gates` (float32 [rows, heads, 2]: decay, write strength) replace w where gates are per head."""
+    lib = _lib("core")
+    for t, what in ((q, "queries"), (k, "keys"), (w, "decays"), (v, "values")):
+        if t is not None and (t.dtype != torch.float32 or not t.is_cuda or t.stride(-1) != 1):
+            raise KernelError(f"gated_scan: the {what} are not float32 rows on the GPU")
+    if gates is not None:
+        _need(gates, torch.float32, "gates")
+    a = _gated_arg(g, o, nq, state, seq_first_row, seq_slot)
+    a.q, a.k, a.w, a.v, a.gates = _ptr(q), _ptr(k), _ptr(w), _ptr(v), _ptr(gates)
+    a.q_ld, a.k_ld, a.w_ld, a.v_ld = q.stride(0), k.stride(0), 0 if w is None else w.stride(0), v.stride(0)
+    _check(lib, lib.x0ne_gated_scan(a, n_seqs, _stream()), "gated_scan")
+
+
+def gated_step(g: GatedState, raw: GatedRawArg, o: torch.Tensor, nq: Optional[torch.Tensor], state: torch.Tensor, seq_first_row: torch.Tensor,
+               seq_slot: torch.Tensor, n_seqs: int) -> None:
+    """Gates and one token's step of every sequence (each brings one row): the bits of the gates' kernels and the scan."""
+    lib = _lib("core")
+    a = _gated_arg(g, o, nq, state, seq_first_row, seq_slot)
+    _check(lib, lib.x0ne_gated_step(a, raw, n_seqs, _stream()), "gated_step")
+
+
+def channel_gates(raw: GatedRawArg, out: torch.Tensor, n_rows: int, channels: int) -> None:
+    """out[r] = [silu(q) | 1 - f | f], f = lower + (1 - lower) sigmoid(z + bias), float32 [rows, 3 * channels]."""
+    lib = _lib("core")
+    _need(out, torch.float32, "gates")
+    if out.shape[-1] != 3 * channels or out.numel() < n_rows * 3 * channels:
+        raise KernelError("channel_gates: the output does not hold three values per channel")
+    _check(lib, lib.x0ne_channel_gates(raw, _ptr(out), n_rows, channels, _stream()), "channel_gates")
+
+
+def head_gates(g: GatedState, raw: GatedRawArg, gates: torch.Tensor, state: torch.Tensor, seq_first_row: torch.Tensor, seq_slot: torch.Tensor,
+               n_seqs: int) -> None:
+    """Decay and write strength of every (row, head), [rows, heads, 2], with the running maximum carried in the state."""
+    lib = _lib("core")
+    _need(gates, torch.float32, "gates")
+    _need(state, torch.float32, "state")
+    _check(lib, lib.x0ne_head_gates(raw, _ptr(gates), _ptr(state), state.stride(0), _ptr(seq_first_row), _ptr(seq_slot), n_seqs, g.heads,
+                                    _stream()), "head_gates")
+
+
+def scan_head_norm(o: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, out_col: int, n_rows: int, heads: int, v_dim: int, eps: float,
+                   nq: Optional[torch.Tensor] = None, em: Optional[torch.Tensor] = None, q_scale: float = 1.0, tiny: float = 0.0,
+                   gate: Optional[torch.Tensor] = None, post: float = 1.0) -> None:
+    """out[row, out_col + ...] = y / sqrt(mean(y^2) + eps) * weight [* sigmoid(gate)] * post per head, with y = o, or with `nq`
+    y = q_scale o / (max(|q_scale nq|, em) + tiny).  `weight`: v_dim values for all heads, or one per (head, value); `gate`: a
+    float32 view of heads * v_dim columns."""
+    lib = _lib("core")
+    for t, what in ((o, "scan output"), (weight, "head norm weight"), (nq, "key sums"), (em, "maxima")):
+        if t is not None:
+            _need(t, torch.float32, what)
+    _need(out, out.dtype, "normed heads")
+    hv = heads * v_dim
+    if o.shape[-1] != hv or weight.numel() not in (v_dim, hv) or out_col < 0 or out_col + hv > out.shape[-1] or out.numel() < n_rows * out.shape[-1]:
+        raise KernelError("scan_head_norm: shapes do not match")
+    if gate is not None and (gate.dtype != torch.float32 or not gate.is_cuda or gate.shape[-1] != hv or gate.stride(-1) != 1):
+        raise KernelError("scan_head_norm: the gate is not a float32 view of the heads' values")
+    arg = HeadNormArg(_ptr(o), _ptr(nq), _ptr(em), float(q_scale), float(tiny), _ptr(weight), 1 if weight.numel() == v_dim and heads > 1 else 0,
+                      _ptr(gate), gate.stride(0) if gate is not None else 0, float(eps), float(post), out.shape[-1], heads, v_dim)
+    _check(lib, lib.x0ne_scan_head_norm(arg, out.data_ptr() + out_col * out.element_size(), dtype_tag(out.dtype), n_rows, _stream()),
+           "scan_head_norm")

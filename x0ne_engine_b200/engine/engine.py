@@ -99,7 +99,7 @@ class Engine:
         self.vocab_size = spec.vocab_size
         needs = self.model.cache_needs()
         self.cache = SequenceCache(needs, [e.reads_cache_of for e in spec.run_order], max_tokens, self.max_seq_len,
-                                   self.dtype, self.device, max_slots=max_slots)
+                                   self.dtype, self.device, max_slots=max_slots, model_needs=self.model.model_cache_needs())
         self.max_step_tokens = int(max_step_tokens or min(8192, max(PAGE_SIZE, max_tokens)))
         self.ws = Workspace(self.max_step_tokens, self.device)
         self.ws.max_want = self.max_step_tokens

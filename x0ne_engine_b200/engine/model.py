@@ -57,14 +57,22 @@ def optional_duplicates_of_spec(spec: ModelSpec) -> Dict[str, str]:
     return dict(P.HEADS.get(spec.head.kind).optional_duplicates(spec.head))
 
 
-def cache_need_of_layer(layer: LayerSpec) -> P.CacheNeed:
-    """What a run-order entry of this layer keeps per sequence: its mixer's need.  A layer without
-    a mixer keeps nothing; a layer may hold one mixer that keeps something."""
-    needs = [cls.cache_need(ps) for _, cls, ps in layer_part_classes(layer) if issubclass(cls, P.Mixer)]
-    needs = [n for n in needs if n.kind != "none"]
-    if len(needs) > 1:
-        raise ConfigError("a layer with two mixers that both keep something per sequence is not served: "
+def cache_needs_of_layer(layer: LayerSpec) -> List[P.CacheNeed]:
+    """Everything a run-order entry of this layer keeps per sequence, of all its parts: keys and values once at most, states
+    told apart by their tags."""
+    needs = [n for _, cls, ps in layer_part_classes(layer) for n in cls.cache_needs(ps) if n.kind != "none"]
+    states = [n.tag for n in needs if n.kind == "state"]
+    if sum(n.kind == "kv" for n in needs) > 1 or len(set(states)) != len(states):
+        raise ConfigError("a layer with two mixers that both keep keys and values, or states of one tag, is not served: "
                           "give each a layer of its own")
+    return needs
+
+
+def cache_need_of_layer(layer: LayerSpec) -> P.CacheNeed:
+    """The one thing a run-order entry of this layer keeps per sequence (a CacheNeed of kind "none" where it keeps nothing)."""
+    needs = cache_needs_of_layer(layer)
+    if len(needs) > 1:
+        raise ConfigError("this layer keeps several things per sequence")
     return needs[0] if needs else P.CacheNeed()
 
 
@@ -85,9 +93,11 @@ def step_bytes_of_spec(spec: ModelSpec, dtype_bytes: int = 2):
     for e in spec.run_order:
         layer = spec.layers[e.layer]
         weights += sum(nbytes(n) for _, cls, ps in layer_part_classes(layer) for n in cls.tensor_needs(ps))
-        need = cache_need_of_layer(layer)
-        if need.kind == "kv" and e.reads_cache_of is None:
-            cache += need.kv_heads * (need.head_dim + (need.head_dim if need.v_dim is None else need.v_dim)) * dtype_bytes
+        if e.before is not None:
+            weights += sum(nbytes(n) for n in P.OPENERS.get(e.before.kind).tensor_needs(e.before) if n.role == "matrix" and n.init == "linear")
+        for need in cache_needs_of_layer(layer):
+            if need.kind == "kv" and e.reads_cache_of is None:
+                cache += need.kv_heads * (need.head_dim + (need.head_dim if need.v_dim is None else need.v_dim)) * dtype_bytes
     return weights, cache
 
 
@@ -123,9 +133,13 @@ class CausalLM:
         and that it takes padding rows (see `parts.Part.replayable`)."""
         return all(p.replayable for p in self.parts()) and all(b.replayable for b in self.blocks)
 
-    def cache_needs(self) -> List[P.CacheNeed]:
-        """One CacheNeed per run-order entry."""
-        return [cache_need_of_layer(self.spec.layers[e.layer]) for e in self.spec.run_order]
+    def cache_needs(self) -> List[List[P.CacheNeed]]:
+        """The CacheNeeds of every run-order entry."""
+        return [cache_needs_of_layer(self.spec.layers[e.layer]) for e in self.spec.run_order]
+
+    def model_cache_needs(self) -> List[P.CacheNeed]:
+        """What the model keeps per sequence outside its layers."""
+        return list(type(self.embedding).cache_needs(self.spec.embedding))
 
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         for part in self.parts():
@@ -136,6 +150,7 @@ class CausalLM:
         total = self.head.weight_bytes()
         for e in self.spec.run_order:
             total += sum(p.weight_bytes() for p in self.blocks[e.layer].parts())
+        total += sum(o.weight_bytes() for o in self.openers if o is not None)
         return total
 
     def forward(self, ctx, want_rows: Optional[torch.Tensor], n_want: int, logits: Optional[torch.Tensor]):

@@ -1,8 +1,8 @@
 """The parts layers are made of, and their registries."""
-from .base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, OPENERS, PART_REGISTRIES, POSITIONS, Block, BuildEnv,
-                   CacheNeed, Embedding, FeedForward, Head, Mixer, Norm, Opener, Part, PositionEncoding, Registry)
+from .base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, INPUT_TRANSFORMS, MIXERS, NORMS, OPENERS, PART_REGISTRIES, POSITIONS, Block, BuildEnv,
+                   CacheNeed, Embedding, FeedForward, Head, InputTransform, Mixer, Norm, Opener, Part, PositionEncoding, Registry)
 from .linear import Linear
-from . import attention, block, diff_attention, distance_attention, embedding, latent_attention, masked_attention, mlp, moe, norm, recurrent, rope, selective_scan, window_attention  # noqa: F401  (registers the built-in parts)
+from . import attention, block, diff_attention, distance_attention, embedding, gated_recurrence, input_conv, latent_attention, masked_attention, mlp, moe, norm, recurrent, rope, selective_scan, side_by_side, sigmoid_attention, window_attention  # noqa: F401  (registers the built-in parts)
 from .attention import GQAttention
 from .block import ParallelBlock, PreNormBlock, PreNormMixerBlock, SandwichBlock
 from .latent_attention import LatentAttention
@@ -10,7 +10,11 @@ from .masked_attention import MaskedAttention
 from .distance_attention import DistanceBiasAttention
 from .diff_attention import DifferentialAttention
 from .selective_scan import SelectiveScan
-from .embedding import LMHead, PassOpener, TokenEmbedding
+from .embedding import ConcatOpener, LMHead, PassOpener, SumEmbedding, TokenEmbedding
+from .gated_recurrence import ChannelGatedRecurrence, MatrixMemory
+from .input_conv import CausalInputConv
+from .side_by_side import ProjectedMixer, SideBySide
+from .sigmoid_attention import SigmoidAttention
 from .mlp import BiasedMLP, ClippedGLU, SwiGLU
 from .recurrent import MatrixStateRecurrence
 from .moe import RoutedExperts
@@ -21,5 +25,6 @@ from .rope import NoPosition, Rope, YarnRope, inv_freq_f32, yarn_frequencies
 __all__ = ["BLOCKS", "EMBEDDINGS", "FEED_FORWARDS", "HEADS", "MIXERS", "NORMS", "PART_REGISTRIES", "POSITIONS", "Block",
            "BuildEnv", "CacheNeed", "Embedding", "FeedForward", "Head", "Mixer", "Norm", "Part", "PositionEncoding",
            "Registry", "Linear", "GQAttention", "OPENERS", "Opener", "PassOpener", "DistanceBiasAttention", "BiasedMLP",
-           "MatrixStateRecurrence", "PreNormMixerBlock", "DifferentialAttention", "SelectiveScan",
+           "MatrixStateRecurrence", "PreNormMixerBlock", "ConcatOpener", "SumEmbedding", "ChannelGatedRecurrence", "MatrixMemory", "CausalInputConv",
+           "InputTransform", "INPUT_TRANSFORMS", "ProjectedMixer", "SideBySide", "SigmoidAttention", "DifferentialAttention", "SelectiveScan",
            "PreNormBlock", "ParallelBlock", "SandwichBlock", "SinkWindowAttention", "RoutedExperts", "PostNormed", "MaskedAttention", "LatentAttention", "ClippedGLU", "YarnRope", "yarn_frequencies", "LMHead", "TokenEmbedding", "SwiGLU", "RMSNorm", "NoPosition", "Rope", "inv_freq_f32"]

@@ -21,6 +21,9 @@ sees the model's name or its config.json.  The kinds:
                      delta)` returns the pending delta.
   * `Embedding`    — `forward(ctx, resid, n_rows)` fills the float32 residual from the token ids.
   * `Head`         — `forward(normed, logits, n_rows)` writes float32 logits of the normed rows.
+  * `InputTransform` — `forward(ctx, entry, norm, resid, delta, n_rows)`: stands between a sublayer's norm and its mixer: adds
+                     the pending delta and norms the residual through `norm` (so that it may do both in one launch) and
+                     returns the rows the mixer reads.  It may keep something per sequence (`cache_needs`).
   * `Opener`       — `forward(ctx, resid, delta, n_rows)`: runs right before a run-order entry that names one
                      (`RunEntry.before`); adds the pending delta and whatever it brings into the residual.
 
@@ -47,6 +50,9 @@ class CacheNeed:
     last `window` of them.  `v_dim` is the width of a value row where it differs from the keys'
     (None: the same; 0: no values are kept, the mixer reads them out of its keys).  kind "state": a float32 array of `state_shape` per sequence, zero
     when the sequence starts.  kind "none": nothing.
+
+    `tag` tells apart the states that the parts of one layer keep (a mixer's own, an input transform's, those of two mixers
+    side by side); a part reads its own through `ctx.cache.state(entry, tag)`.
     """
     kind: str = "none"
     kv_heads: int = 0
@@ -54,6 +60,7 @@ class CacheNeed:
     window: Optional[int] = None
     state_shape: Tuple[int, ...] = ()
     v_dim: Optional[int] = None
+    tag: str = ""
 
 
 @dataclass
@@ -82,6 +89,11 @@ class Part:
     def tensor_needs(spec: PartSpec) -> List[TensorNeed]:
         return []
 
+    @classmethod
+    def cache_needs(cls, spec: PartSpec) -> List[CacheNeed]:
+        """Everything the part keeps per sequence, for every run-order entry of its layer (an embedding: for the model)."""
+        return []
+
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         """Receives the device tensors named in `tensor_needs`."""
 
@@ -100,14 +112,26 @@ class Mixer(Part):
     def cache_need(spec: PartSpec) -> CacheNeed:
         return CacheNeed()
 
+    @classmethod
+    def cache_needs(cls, spec: PartSpec) -> List[CacheNeed]:
+        need = cls.cache_need(spec)
+        return [need] if need.kind != "none" else []
+
     def forward(self, ctx, entry: int, x: torch.Tensor, n_rows: int, cache_entry: Optional[int] = None,
                 write_cache: bool = True) -> torch.Tensor:
+        raise NotImplementedError
+
+
+class InputTransform(Part):
+    def forward(self, ctx, entry: int, norm: "Norm", resid: torch.Tensor, delta, n_rows: int) -> torch.Tensor:
         raise NotImplementedError
 
 
 class FeedForward(Part):
     out_buffer = "delta"        # the workspace buffer the result goes to; an arrangement that runs the
                                 # feed-forward beside the mixer names another one
+    defer_bias = False          # True: the arrangement adds `result_bias` (if there is one) itself, where it adds the result
+    result_bias: Optional[torch.Tensor] = None
 
     def forward(self, ctx, x: torch.Tensor, n_rows: int) -> torch.Tensor:
         raise NotImplementedError
@@ -208,6 +232,7 @@ POSITIONS = Registry("position encoding")
 BLOCKS = Registry("block")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
+INPUT_TRANSFORMS = Registry("input transform")
 OPENERS = Registry("opener")
 # the registry behind each kind of part a block's role may name
-PART_REGISTRIES = {"norm": NORMS, "mixer": MIXERS, "feed_forward": FEED_FORWARDS}
+PART_REGISTRIES = {"norm": NORMS, "mixer": MIXERS, "feed_forward": FEED_FORWARDS, "input_transform": INPUT_TRANSFORMS}

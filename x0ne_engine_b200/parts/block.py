@@ -57,26 +57,33 @@ class SandwichBlock(Block):
     """x += post_norm(mixer(norm(x))); x += post_norm(ffn(norm(x))): every sublayer has a norm before it and one
     after it, on its result, before the add.  The normed result is never stored: the result travels with its
     norm (`PostNormed`) to the next norm in line, whose kernel norms it, adds it to the float32 residual
-    and norms the sum.  A layer may leave the feed-forward (and its two norms) out."""
+    and norms the sum.  A layer may leave the feed-forward (and its two norms) out.  With `mixer_input` an input transform
+    stands between the first norm and the mixer.  A feed-forward's result bias travels with its result."""
     replayable = True
-    ROLES = {"mixer_norm": "norm", "mixer": "mixer", "mixer_post_norm": "norm", "ffn_norm": "norm", "ffn": "feed_forward",
-             "ffn_post_norm": "norm"}
-    OPTIONAL = ("ffn_norm", "ffn", "ffn_post_norm")
+    ROLES = {"mixer_norm": "norm", "mixer_input": "input_transform", "mixer": "mixer", "mixer_post_norm": "norm", "ffn_norm": "norm",
+             "ffn": "feed_forward", "ffn_post_norm": "norm"}
+    OPTIONAL = ("mixer_input", "ffn_norm", "ffn", "ffn_post_norm")
 
     def __init__(self, parts):
         super().__init__(parts)
         if (self.ffn is None) != (self.ffn_norm is None) or (self.ffn is None) != (self.ffn_post_norm is None):
             raise ValueError("a sandwich layer has its feed-forward with both of its norms, or none of the three")
+        if self.ffn is not None:
+            self.ffn.defer_bias = True
 
     def forward(self, ctx, entry, resid, delta, cache_entry=None, write_cache=True):
         normed = ctx.ws.buffer("normed", (ctx.ws.max_rows, resid.shape[-1]), ctx.dtype)
-        self.mixer_norm.add_norm(ctx, resid, delta, normed, ctx.n_rows)
-        mixed = PostNormed(self.mixer.forward(ctx, entry, normed, ctx.n_rows, cache_entry=cache_entry, write_cache=write_cache),
+        if self.mixer_input is not None:
+            read = self.mixer_input.forward(ctx, entry, self.mixer_norm, resid, delta, ctx.n_rows)
+        else:
+            self.mixer_norm.add_norm(ctx, resid, delta, normed, ctx.n_rows)
+            read = normed
+        mixed = PostNormed(self.mixer.forward(ctx, entry, read, ctx.n_rows, cache_entry=cache_entry, write_cache=write_cache),
                            self.mixer_post_norm)
         if self.ffn is None:
             return mixed
         self.ffn_norm.add_norm(ctx, resid, mixed, normed, ctx.n_rows)
-        return PostNormed(self.ffn.forward(ctx, normed, ctx.n_rows), self.ffn_post_norm)
+        return PostNormed(self.ffn.forward(ctx, normed, ctx.n_rows), self.ffn_post_norm, self.ffn.result_bias)
 
 
 BLOCKS.register("prenorm", PreNormBlock)

@@ -16,8 +16,11 @@ from .linear import Linear
 class SwiGLU(FeedForward):
     """down( silu(gate x) * up x ): one product on the packed [gate; up] weight (gate rows, then
     up rows: x0ne-core/runtime/src/weights.rs:218-219), the activation
-    g / (1 + expf(-g)) * u (x0ne-core/kernels/cuda/swiglu.cu:5-11), one product with down.
-    Parameters: hidden_size, intermediate_size, names.{gate, up, down}."""
+    g / (1 + expf(-g)) * u (x0ne-core/kernels/cuda/swiglu.cu:5-11), one product with down.  With `bias` every projection has
+    one: the gate's and the up branch's are added in float32 ahead of the activation (in the products' epilogues where
+    those have the activation); the down projection's is added where the result joins the residual if the arrangement
+    does that (`defer_bias`), else behind the product.
+    Parameters: hidden_size, intermediate_size, bias (default False), names.{gate, up, down, gate_bias, up_bias, down_bias}."""
     replayable = True
 
     def __init__(self, spec, env):
@@ -26,16 +29,26 @@ class SwiGLU(FeedForward):
         self.inter = int(spec["intermediate_size"])
         self.gate_up = None
         self.down = None
+        self.biased = bool(spec.get("bias"))
+        self.gate_up_bias = self.down_bias = None
 
     @staticmethod
     def tensor_needs(spec: PartSpec) -> List[TensorNeed]:
         h, i, n = int(spec["hidden_size"]), int(spec["intermediate_size"]), spec["names"]
-        return [TensorNeed(n["gate"], (i, h)), TensorNeed(n["up"], (i, h)), TensorNeed(n["down"], (h, i))]
+        needs = [TensorNeed(n["gate"], (i, h)), TensorNeed(n["up"], (i, h)), TensorNeed(n["down"], (h, i))]
+        if spec.get("bias"):
+            needs += [TensorNeed(n["gate_bias"], (i,), role="vector", init="linear"), TensorNeed(n["up_bias"], (i,), role="vector", init="linear"),
+                      TensorNeed(n["down_bias"], (h,), role="vector", init="linear")]
+        return needs
 
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         n = self.spec["names"]
         self.gate_up = Linear(torch.cat([tensors[n["gate"]], tensors[n["up"]]], dim=0).contiguous())
         self.down = Linear(tensors[n["down"]])
+        if self.biased:
+            self.gate_up_bias = torch.cat([tensors[n["gate_bias"]], tensors[n["up_bias"]]]).contiguous()
+            self.down_bias = tensors[n["down_bias"]]
+            self.result_bias = self.down_bias if self.defer_bias else None
 
     def weight_bytes(self) -> int:
         return self.gate_up.weight_bytes() + self.down.weight_bytes()
@@ -46,15 +59,17 @@ class SwiGLU(FeedForward):
         out = ctx.ws.buffer(self.out_buffer, (ctx.ws.max_rows, self.hidden), self.env.dtype)
         kernel = ops.product_kernel(self.gate_up.weight, n_rows, fused=True)       # the routing table (csrc/routes.py)
         if kernel == "skinny":
-            ops.gemm_bf16_skinny_tcgen05(x, self.gate_up.weight, act, n_rows, swiglu=True)   # 9 to 64 rows, tcgen05
+            ops.gemm_bf16_skinny_tcgen05(x, self.gate_up.weight, act, n_rows, swiglu=True, bias=self.gate_up_bias)   # 9 to 64 rows, tcgen05
         elif kernel == "smallm":
-            ops.gemm_bf16_smallm(x, self.gate_up.weight, act, n_rows, swiglu=True)     # activation in the epilogue
+            ops.gemm_bf16_smallm(x, self.gate_up.weight, act, n_rows, swiglu=True, bias=self.gate_up_bias)     # activation in the epilogue
         elif kernel == "tc_pair":
-            ops.gemm_bf16_tcgen05(x, self.gate_up.weight, act, n_rows, swiglu=True)    # tcgen05, activation in the epilogue
+            ops.gemm_bf16_tcgen05(x, self.gate_up.weight, act, n_rows, swiglu=True, bias=self.gate_up_bias)    # tcgen05, activation in the epilogue
         else:
             self.gate_up(x, gu, n_rows)
-            ops.swiglu(gu, act, n_rows)
+            ops.swiglu(gu, act, n_rows, self.gate_up_bias)
         self.down(act, out, n_rows)
+        if self.down_bias is not None and not self.defer_bias:
+            ops.bias_act(out, self.down_bias, out, n_rows)
         return out
 
 
