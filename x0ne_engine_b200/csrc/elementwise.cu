@@ -964,15 +964,12 @@ X0NE_API int x0ne_embed_sum(EmbedSumArgs a, int dt, int n_rows, cudaStream_t str
 // ----------------------------------------------------------------------------------------
 // The operand of a product over two concatenated rows:  out[r] = [ x | x0[r] ]  with
 //   x = resid[r] + norm(delta[r] + bias_d) * w_d      (delta null: resid alone; w_d null: delta added as it is)
-// in float32, rounded once to the activation type.  The residual is only read.  With `lo` (bfloat16 runs) the rows n_rows
-// .. 2 n_rows - 1 of out receive what that rounding lost, rounded in turn: the product over both, added up, sees the
-// float32 values to 16 bits.
+// in float32, rounded once to the activation type.  The residual is only read (the product's result replaces it).
 // One block per row; the sum of squares is a fixed-order block sum.
 // ----------------------------------------------------------------------------------------
 template <typename T>
 __global__ void concat_rows_kernel(const float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ bias_d,
-                                   const float* __restrict__ w_d, float eps_d, const float* __restrict__ x0, T* __restrict__ out, int n_rows,
-                                   int hidden, int lo) {
+                                   const float* __restrict__ w_d, float eps_d, const float* __restrict__ x0, T* __restrict__ out, int hidden) {
     __shared__ float sh[32];
     pdl_prologue();
     const int64_t row = blockIdx.x;
@@ -980,7 +977,6 @@ __global__ void concat_rows_kernel(const float* __restrict__ resid, const T* __r
     const float* z = x0 + row * hidden;
     const T* d = delta != nullptr ? delta + row * hidden : nullptr;
     T* o = out + row * 2 * hidden;
-    T* l = lo ? out + (row + n_rows) * 2 * hidden : nullptr;
     float scale = 1.f;
     if (d != nullptr && w_d != nullptr) {
         float ss = 0.f;
@@ -993,40 +989,20 @@ __global__ void concat_rows_kernel(const float* __restrict__ resid, const T* __r
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         float v = r[i];
         if (d != nullptr) v += (to_f32(d[i]) + (bias_d != nullptr ? bias_d[i] : 0.f)) * scale * (w_d != nullptr ? w_d[i] : 1.f);
-        const float w = z[i];
-        const T hv = from_f32<T>(v), hw = from_f32<T>(w);
-        o[i] = hv;
-        o[hidden + i] = hw;
-        if (l != nullptr) {
-            l[i] = from_f32<T>(v - to_f32(hv));
-            l[hidden + i] = from_f32<T>(w - to_f32(hw));
-        }
+        o[i] = from_f32<T>(v);
+        o[hidden + i] = from_f32<T>(z[i]);
     }
 }
 
-// out[i] = a[i] + b[i], float32 (the two halves of such a product)
-__global__ void add_f32_kernel(const float* __restrict__ a, const float* __restrict__ b, float* __restrict__ out, int64_t total) {
-    pdl_prologue();
-    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) out[i] = a[i] + b[i];
-}
-
 X0NE_API int x0ne_concat_rows(const float* resid, const void* delta, int dt, const float* bias_d, const float* w_d, float eps_d, const float* x0,
-                              void* out, int n_rows, int hidden, int lo, cudaStream_t stream) {
+                              void* out, int n_rows, int hidden, cudaStream_t stream) {
     X0NE_REQUIRE(n_rows >= 0 && hidden > 0 && resid != nullptr && x0 != nullptr && out != nullptr, "concat_rows: rows %d hidden %d", n_rows, hidden);
     X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "concat_rows: unknown dtype tag %d", dt);
     if (n_rows == 0) return 0;
     const int block = hidden >= 512 ? 512 : (hidden + 31) / 32 * 32;
     if (dt == X0NE_F32)
-        x0ne_launch(concat_rows_kernel<float>, dim3(n_rows), dim3(block), 0, stream, resid, (const float*)delta, bias_d, w_d, eps_d, x0, (float*)out, n_rows, hidden, lo);
+        x0ne_launch(concat_rows_kernel<float>, dim3(n_rows), dim3(block), 0, stream, resid, (const float*)delta, bias_d, w_d, eps_d, x0, (float*)out, hidden);
     else
-        x0ne_launch(concat_rows_kernel<bf16>, dim3(n_rows), dim3(block), 0, stream, resid, (const bf16*)delta, bias_d, w_d, eps_d, x0, (bf16*)out, n_rows, hidden, lo);
-    X0NE_LAUNCH_CHECK();
-}
-
-X0NE_API int x0ne_add_f32(const float* a, const float* b, float* out, int64_t total, cudaStream_t stream) {
-    X0NE_REQUIRE(total >= 0 && a != nullptr && b != nullptr && out != nullptr, "add_f32: %lld values", (long long)total);
-    if (total == 0) return 0;
-    const int64_t blocks = (total + 255) / 256;
-    x0ne_launch(add_f32_kernel, dim3((unsigned)(blocks < 148 * 64 ? blocks : 148 * 64)), dim3(256), 0, stream, a, b, out, total);
+        x0ne_launch(concat_rows_kernel<bf16>, dim3(n_rows), dim3(block), 0, stream, resid, (const bf16*)delta, bias_d, w_d, eps_d, x0, (bf16*)out, hidden);
     X0NE_LAUNCH_CHECK();
 }

@@ -157,8 +157,7 @@ _SIGNATURES = {
     "x0ne_scan_head_norm": [HeadNormArg, _P, _I, _I, _P],
     "x0ne_head_norm_rope_kv_write": [HeadRopeArg, _P, _I, None, _P],
     "x0ne_embed_sum": [EmbedSumArg, _I, _I, _P],
-    "x0ne_concat_rows": [_P, _P, _I, _P, _P, _F, _P, _P, _I, _I, _I, _P],
-    "x0ne_add_f32": [_P, _P, _P, _L, _P],
+    "x0ne_concat_rows": [_P, _P, _I, _P, _P, _F, _P, _P, _I, _I, _P],
     "x0ne_input_conv": [_P, _I, _P, _P, _L, _L, _P, _P, _P, _I, _I, _I, _I, _P],
     "x0ne_norm_conv_step": [NormConvArg, _P, _I, _I, _P],
     "x0ne_add_normed_rmsnorm": [_P, _P, _P, _P, _F, _P, _P, _I, _P, _I, _I, _F, _P],
@@ -1450,9 +1449,9 @@ def embed_sum(table: torch.Tensor, pairs: Optional[torch.Tensor], positions: Opt
 
 
 def concat_rows(resid: torch.Tensor, delta: Optional[torch.Tensor], delta_bias: Optional[torch.Tensor], delta_weight: Optional[torch.Tensor],
-                delta_eps: float, x0: torch.Tensor, out: torch.Tensor, n_rows: int, lo: bool = False) -> None:
+                delta_eps: float, x0: torch.Tensor, out: torch.Tensor, n_rows: int) -> None:
     """out[r] = [x | x0[r]] with x = resid[r] + rmsnorm(delta[r] + delta_bias) * delta_weight (no weight: delta is added as it
-    is; no delta: resid alone), rounded once to out's type; `lo`: rows n_rows .. 2 n_rows - 1 receive what that lost."""
+    is; no delta: resid alone), rounded once to out's type."""
     lib = _lib("core")
     _need(resid, torch.float32, "residual")
     _need(x0, torch.float32, "second rows")
@@ -1463,20 +1462,10 @@ def concat_rows(resid: torch.Tensor, delta: Optional[torch.Tensor], delta_bias: 
     for t, what in ((delta_bias, "delta bias"), (delta_weight, "norm weight of the delta")):
         if t is not None:
             _need(t, torch.float32, what)
-    if out.shape[-1] != 2 * hidden or out.numel() < (2 if lo else 1) * n_rows * 2 * hidden or x0.numel() < n_rows * hidden or resid.numel() < n_rows * hidden:
+    if out.shape[-1] != 2 * hidden or out.numel() < n_rows * 2 * hidden or x0.numel() < n_rows * hidden or resid.numel() < n_rows * hidden:
         raise KernelError("concat_rows: shapes do not match")
     _check(lib, lib.x0ne_concat_rows(_ptr(resid), _ptr(delta), dtype_tag(out.dtype), _ptr(delta_bias), _ptr(delta_weight), float(delta_eps),
-                                     _ptr(x0), _ptr(out), n_rows, hidden, 1 if lo else 0, _stream()), "concat_rows")
-
-
-def add_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, total: int) -> None:
-    """out[i] = a[i] + b[i] for the first `total` values."""
-    lib = _lib("core")
-    for t in (a, b, out):
-        _need(t, torch.float32, "float32 rows")
-        if t.numel() < total:
-            raise KernelError("add_f32: fewer values than asked for")
-    _check(lib, lib.x0ne_add_f32(_ptr(a), _ptr(b), _ptr(out), total, _stream()), "add_f32")
+                                     _ptr(x0), _ptr(out), n_rows, hidden, _stream()), "concat_rows")
 
 
 INPUT_CONV_MAX_TAPS = 17

@@ -87,8 +87,7 @@ class ConcatOpener(Opener):
     """The start of a pass over a repeated stretch of layers: the residual becomes W [x; x0], x being the residual with the
     pending result of the layer before and x0 the embedding output (`EMBEDDING_OUTPUT`, left there by the embedding).  The
     product's operand is built by one launch (which also norms and adds the pending result), its float32 result is the new
-    residual.  A bfloat16 run gives the product the operand as two rows, its bfloat16 and the bfloat16 of what that
-    rounding lost, and adds the two results, so that the residual does not lose its small digits here.
+    residual.
     Parameters: hidden_size, names.weight ([hidden_size, 2 hidden_size])."""
     replayable = True
 
@@ -117,16 +116,10 @@ class ConcatOpener(Opener):
             raise ValueError("a concatenating opener takes the pending result of a layer as one tensor")
         if norm is not None and norm.groups != 1:
             raise ValueError("a norm in groups does not take a result that is still to be normed")
-        halves = 2 if dt == torch.bfloat16 else 1
         x0 = ws.buffer(EMBEDDING_OUTPUT, (ws.max_rows, h), torch.float32)
-        cat = ws.buffer("opener.rows", (halves * ws.max_rows, 2 * h), dt)
-        ops.concat_rows(resid, delta, bias, None if norm is None else norm.weight, 0.0 if norm is None else norm.eps, x0, cat, n_rows, lo=halves == 2)
-        if halves == 1:
-            self.w(cat, resid, n_rows)
-        else:
-            out = ws.buffer("opener.out", (halves * ws.max_rows, h), torch.float32)
-            self.w(cat, out, halves * n_rows)
-            ops.add_f32(out, out[n_rows:], resid, n_rows * h)
+        cat = ws.buffer("opener.rows", (ws.max_rows, 2 * h), dt)
+        ops.concat_rows(resid, delta, bias, None if norm is None else norm.weight, 0.0 if norm is None else norm.eps, x0, cat, n_rows)
+        self.w(cat, resid, n_rows)
         return None
 
 
