@@ -13,9 +13,9 @@ time); `e2e` is the same rate through `Model.generate` with host token lists in 
 and 64 and the milliseconds a 128-token and a 512-token prompt take through the step function; `roofline` places the decode step against the bytes it must read.  One JSON line is
 printed.  This library runs on one GPU: for --gpus above 1 a line says so and the exit code is 2.
 
-    python bench.py --design rovurax|tenetar|retuvik|barorax [--sizes 1.7b,8b] [--layers 8] [--chunk 1024] [--steps K]
+    python bench.py --design rovurax|tenetar|retuvik|barorax|ravapel [--sizes 1.7b,8b] [--layers 8] [--chunk 1024] [--steps K]
 
-instead runs that design beside Qwen3 (retuvik: beside Tenetar; barorax: beside Retuvik) at equal sizes (random bfloat16 weights, the same engine,
+instead runs that design beside Qwen3 (retuvik: beside Tenetar; barorax and ravapel: beside Retuvik) at equal sizes (random bfloat16 weights, the same engine,
 step function and decode graphs): one prompt of --prefill-tokens through the step function, then decode
 at --batch, device-timed; one JSON line with a row per size and design.
 """
@@ -217,6 +217,24 @@ def barorax_config(size: dict, layers: int, vocab: int, chunk: int):
                              "loop": {"start": 0, "stop": layers, "times": 1}})
 
 
+def ravapel_config(size: dict, layers: int, vocab: int, chunk: int):
+    """A Ravapel configuration of the given layer sizes.  Every other layer is a recurrence with a gate per channel (heads of
+    128 x 128 that fill the width), the rest are attention with sigmoid weights over chunks (rotation over half of every
+    head) beside a matrix memory (half as many heads, keys of half the head size, values of it); every layer has the
+    dense gated feed-forward of the full width with biases, and an input convolution of 4 taps.  The whole list is a
+    stretch that runs once, so a pass opener runs."""
+    from x0ne_engine_b200.config import config_from_dict
+    w, ff, H, G, d = size["width"], size["ff"], size["heads"], size["kv_heads"], size["dim"]
+    rec = {"type": "hgrn2", "mixer": {"dim": 128, "heads": w // 128, "vdim": 128}}
+    par = {"type": "parallel", "mixer": {
+        "left": {"dim": d, "heads": H, "kv_heads": G, "vdim": d, "scale": d ** -0.5, "mask": {"size": chunk}, "rot": {"base": 10000.0, "dims": d // 2}},
+        "right": {"dim": d // 2, "heads": H // 2, "vdim": d, "gate_cap": 15.0}, "left_scale": 1.0, "right_scale": 1.0}}
+    return config_from_dict({"architecture": "Ravapel", "vocab": vocab, "width": w, "norm": {"eps": 1e-6}, "canon": {"taps": 4},
+                             "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1009, "mul_cur": 9176}}, "max_positions": 16384,
+                             "layers": [{**(par if i % 2 else rec), "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)],
+                             "loop": {"start": 0, "stop": layers, "times": 1}})
+
+
 def design_configs(size: dict, layers: int, vocab: int, chunk: int, design: str = "rovurax"):
     """(the design's configuration, Qwen3 configuration) with the same width, heads, feed-forward, depth and
     vocabulary.  Of every four Rovurax layers three are chunk-masked attention with blended values and
@@ -233,6 +251,8 @@ def design_configs(size: dict, layers: int, vocab: int, chunk: int, design: str 
         return retuvik_config(size, layers, vocab, chunk), tenetar_config(size, layers, vocab, chunk)
     if design == "barorax":        # beside Retuvik: a recurrent mixer with a state, attention over a bounded span, gated experts, a stretch
         return barorax_config(size, layers, vocab, chunk), retuvik_config(size, layers, vocab, chunk)
+    if design == "ravapel":        # beside Retuvik: matrix states per head, attention over a bounded span, a repeated stretch
+        return ravapel_config(size, layers, vocab, chunk), retuvik_config(size, layers, vocab, chunk)
     mlp = {"ff": ff, "kind": "dense", "limit": 7.0}
     att = {"type": "attention", "mlp": mlp, "mixer": {"dim": d, "heads": H, "kv_heads": G, "vdim": d, "scale": d ** -0.5,
                                                         "mask": {"size": chunk}, "v_mix": True}}
@@ -259,7 +279,7 @@ def design_bench(args) -> int:
     layers = args.layers or 8
     vocab = 32768
     rows_out = []
-    other = {"retuvik": "tenetar", "barorax": "retuvik"}.get(args.design, "qwen3")
+    other = {"retuvik": "tenetar", "barorax": "retuvik", "ravapel": "retuvik"}.get(args.design, "qwen3")
     for name in args.sizes.split(","):
         size = DESIGN_SIZES[name]
         for design, cfg in zip((args.design, other), design_configs(size, layers, vocab, args.chunk, args.design)):
@@ -333,12 +353,12 @@ def main() -> int:
     ap.add_argument("--prefill-tokens", type=int, default=2048)
     ap.add_argument("--no-points", action="store_true", help="skip decode at batch 1 and 64")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--design", default=None, choices=["rovurax", "tenetar", "retuvik", "barorax"],
-                    help="instead of the default workload: this design beside Qwen3 (retuvik: beside Tenetar; barorax: beside Retuvik) "
+    ap.add_argument("--design", default=None, choices=["rovurax", "tenetar", "retuvik", "barorax", "ravapel"],
+                    help="instead of the default workload: this design beside Qwen3 (retuvik: beside Tenetar; barorax and ravapel: beside Retuvik) "
                          "at equal sizes (prefill and decode)")
     ap.add_argument("--sizes", default="1.7b,8b", help="with --design: which of " + ", ".join(DESIGN_SIZES))
     ap.add_argument("--chunk", type=int, default=1024,
-                    help="with --design: positions per chunk of the masked attention (rovurax, barorax) or of the sliding window (tenetar, retuvik)")
+                    help="with --design: positions per chunk of the masked attention (rovurax, barorax, ravapel) or of the sliding window (tenetar, retuvik)")
     args = ap.parse_args()
     if args.design is not None and args.impl == "ours" and args.gpus == 1:
         return design_bench(args)

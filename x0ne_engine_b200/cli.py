@@ -559,6 +559,101 @@ def cmd_kernel_bench(a) -> int:
         timed(lambda: ops.wkv_scan(r, k, v, z, w0, u, h, o, state, first, slots, B, heads, n, one_token=per == 1),
               rows * hn * (3 * 2 + 4 + 4) + 2 * B * mats * 4, 4.0 * rows * hn * n)
         return 0
+    if a.kernel in ("gated_scan", "gated_step", "channel_gates", "head_gates", "scan_head_norm"):
+        # a gated linear recurrence's own kernels: --batch sequences of --m rows each, --heads heads of --head-dim channels x
+        # --v-dim values; gates per channel, or per head with --gated (one more state column, the keys' sum)
+        B, per, heads, d, hg = a.batch, a.m, a.q_heads, a.head_dim, a.gated
+        vd = a.v_dim or d
+        rows, hd, hv = B * per, heads * d, heads * vd
+        g = ops.GatedState(heads, d, vd, hg)
+        copies = 1
+        src = torch.randn(rows, 2 * hd + hv + 2 * heads, device=dev)
+        state = torch.randn(B, g.floats, device=dev).mul_(0.1)
+        o, nq, em = torch.empty(rows, hv, device=dev), torch.empty(rows, heads, device=dev), torch.empty(rows, heads, device=dev)
+        first = (torch.arange(B + 1, dtype=torch.int32, device=dev) * per).contiguous()
+        slots = torch.arange(B, dtype=torch.int32, device=dev)
+        pos0 = torch.full((B,), 64, dtype=torch.int32, device=dev)
+        wide, narrow = torch.rand(hd, device=dev), torch.rand(heads, device=dev)
+        if hg:
+            raw = ops.gated_raw(src, 0, hd, 2 * hd, narrow, i_col=2 * hd + hv, f_col=2 * hd + hv + heads, i_bias=narrow, cap=15.0, geometry=g, em=em,
+                                seq_pos0=pos0)
+            gates = torch.rand(rows, heads, 2, device=dev)
+        else:
+            raw = ops.gated_raw(src, 0, hd, 2 * hd, wide, lower=wide)
+            gates = torch.rand(rows, 3 * hd, device=dev)
+        nqp, v, states = nq if hg else None, src[:, 2 * hd:2 * hd + hv], 2 * B * g.floats * 4
+        flops = 6.0 * rows * heads * d * g.cols
+        if a.kernel == "gated_scan" and hg:
+            timed(lambda: ops.gated_scan(g, src[:, :hd], src[:, hd:2 * hd], None, v, gates, o, nqp, state, first, slots, B),
+                  rows * (2 * hd + 2 * hv) * 4 + states, flops)
+        elif a.kernel == "gated_scan":
+            timed(lambda: ops.gated_scan(g, gates[:, :hd], gates[:, hd:2 * hd], gates[:, 2 * hd:], v, None, o, nqp, state, first, slots, B),
+                  rows * (3 * hd + 2 * hv) * 4 + states, flops)
+        elif a.kernel == "gated_step":
+            if per != 1:
+                raise SystemExit("gated_step takes one row per sequence: --m 1")
+            timed(lambda: ops.gated_step(g, raw, o, nqp, state, first, slots, B), rows * (2 * hd + 2 * hv) * 4 + states, flops)
+        elif a.kernel == "channel_gates":
+            if hg:
+                raise SystemExit("channel_gates belongs to gates per channel: leave --gated out")
+            timed(lambda: ops.channel_gates(raw, gates, rows, hd), rows * hd * (2 + 3) * 4)
+        elif a.kernel == "head_gates":
+            if not hg:
+                raise SystemExit("head_gates belongs to gates per head: --gated")
+            timed(lambda: ops.head_gates(g, raw, gates, state, first, slots, B), rows * heads * (2 + 3) * 4)
+        else:
+            act = torch.empty(rows, hv, device=dev, dtype=torch.bfloat16)
+            weight = torch.ones(hv if hg else vd, device=dev)
+            em.fill_(1.0), nq.fill_(2.0)
+            extra = dict(nq=nq, em=em, tiny=1e-6, gate=v) if hg else {}
+            timed(lambda: ops.scan_head_norm(o, weight, act, 0, rows, heads, vd, 1e-6, **extra), rows * hv * (4 + 2 + (4 if hg else 0)))
+        return 0
+    if a.kernel in ("input_conv", "norm_conv_step", "concat_rows", "embed_sum"):
+        # --m rows of --n values: the input convolution of one sequence (4 taps); the residual add, norm and convolution of one
+        # row per sequence; the concatenating opener's operand; the summed embedding
+        rows, h, taps = a.m, a.n, 4
+        copies = 1
+        resid, x0 = torch.randn(rows, h, device=dev), torch.randn(rows, h, device=dev)
+        delta = torch.randn(rows, h, device=dev).bfloat16()
+        out = torch.empty_like(delta)
+        w, conv = torch.ones(h, device=dev), torch.randn(taps, h, device=dev)
+        i32 = dict(dtype=torch.int32, device=dev)
+        if a.kernel == "input_conv":
+            state = torch.zeros(1, (taps - 1) * h, device=dev)
+            first, slots = torch.tensor([0, rows], **i32), torch.zeros(1, **i32)
+            timed(lambda: ops.input_conv(delta, conv, state, out, first, slots, 1, rows), rows * h * (2 + 2))
+        elif a.kernel == "norm_conv_step":
+            state, slots = torch.zeros(rows, (taps - 1) * h, device=dev), torch.arange(rows, **i32)
+            timed(lambda: ops.norm_conv_step(resid, delta, w, w, 1e-6, w, 1e-6, conv, state, out, slots, rows),
+                  rows * h * (4 + 4 + 2 + 2 + 2 * 4 * (taps - 1)) + h * 4 * (3 + taps))
+        elif a.kernel == "concat_rows":
+            cat = torch.empty(rows, 2 * h, device=dev, dtype=torch.bfloat16)
+            timed(lambda: ops.concat_rows(resid, delta, w, w, 1e-6, x0, cat, rows), rows * h * (4 + 2 + 4 + 4))
+        else:
+            table, pairs, pos_t = (torch.randn(n, h, device=dev).bfloat16() for n in (32768, 65522, 16384))
+            tokens, row_pos = torch.randint(0, 32768, (rows,), **i32), torch.arange(rows, **i32)
+            first, slots, last = torch.tensor([0, rows], **i32), torch.zeros(rows, **i32), torch.zeros(1, 1, device=dev)
+            timed(lambda: ops.embed_sum(table, pairs, pos_t, tokens, resid, x0, last, 1009, 9176, slots, row_pos, first, 1, rows), rows * h * (3 * 2 + 2 * 4))
+        return 0
+    if a.kernel == "head_norm_rope":
+        # per-head norms with weights, rotation of half of every head, keys and values into the pages, from a float32
+        # projection; --m rows of one sequence
+        from .cache import SequenceCache
+        from .parts.base import CacheNeed
+        rows, qh, kvh, hd = a.m, a.q_heads, a.kv_heads, a.head_dim
+        vd = a.v_dim or hd
+        cache = SequenceCache([CacheNeed("kv", kvh, hd, None, v_dim=None if vd == hd else vd)], [None], rows + 64, rows + 64, torch.bfloat16, dev)
+        slot = cache.acquire(rows)
+        width = (qh + kvh) * hd + kvh * vd
+        src = torch.randn(rows, width, device=dev)
+        q_out = torch.empty(rows, qh * hd, device=dev, dtype=torch.bfloat16)
+        w, freq, table = torch.ones(hd, device=dev), torch.rand(hd // 4, device=dev), torch.rand(rows, hd // 2, device=dev)
+        slots = torch.full((rows,), slot, dtype=torch.int32, device=dev)
+        pos = torch.arange(rows, dtype=torch.int32, device=dev)
+        copies = 1
+        timed(lambda: ops.head_norm_rope_kv_write(src, 0, qh * hd, (qh + kvh) * hd, w, w, 1e-6, freq, table, hd // 2, q_out, qh, cache.kv_view(0),
+                                                  slots, pos, rows), rows * width * (4 + 2))
+        return 0
     if a.kernel in ("ssm_scan", "causal_conv"):
         # the selective state-space mixer's own kernels: --batch sequences of --m rows each, --n channels of --head-dim
         # states, 4 taps; every sequence goes on from its state (m 1: a decode step)

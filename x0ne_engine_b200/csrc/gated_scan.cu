@@ -15,11 +15,11 @@
 // is the same bits however its sequence is cut into passes, whatever else is in a pass and whichever kernel runs.
 #include "common.cuh"
 
-#define GS_WARPS 4
 #define GS_CW 4                         // state columns of a warp
-#define GS_COLS (GS_WARPS * GS_CW)      // of a block
-#define GS_U 4                          // tokens worked on side by side
+#define GS_COLS 16                      // of a block
+#define GS_U 8                          // tokens worked on side by side
 #define GS_STAGES 3
+#define GS_THREADS (GS_COLS / GS_CW * 32)       // working threads of a block
 
 __device__ __forceinline__ float gs_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float gs_silu(float z) { return z / (1.0f + expf(-z)); }
@@ -69,11 +69,11 @@ template <int KI> __device__ __forceinline__ void gs_load_pairs(f32x2 (&r)[KI / 
 }
 
 // One token: the state's step and this lane's share of the results.
-template <int KI>
-__device__ __forceinline__ void gs_step(f32x2 (&S)[KI / 2][GS_CW], const f32x2 (&q)[KI / 2], const f32x2 (&k)[KI / 2],
-                                        const f32x2 (&w)[KI / 2], const f32x2 (&v)[GS_CW], float* acc) {
+template <int KI, int CW>
+__device__ __forceinline__ void gs_step(f32x2 (&S)[KI / 2][CW], const f32x2 (&q)[KI / 2], const f32x2 (&k)[KI / 2], const f32x2 (&w)[KI / 2],
+                                        const f32x2 (&v)[CW], float* acc) {
 #pragma unroll
-    for (int c = 0; c < GS_CW; ++c) {
+    for (int c = 0; c < CW; ++c) {
         f32x2 a = 0ull;
 #pragma unroll
         for (int p = 0; p < KI / 2; ++p) {
@@ -118,10 +118,10 @@ __device__ __forceinline__ void gs_cp4(float* dst, const float* src, bool ok) {
                  : "memory");
 }
 
-template <int KI>
-__device__ __forceinline__ void gs_load_state(f32x2 (&S)[KI / 2][GS_CW], const float* st, int col0, int C, int D, int lane) {
+template <int KI, int CW>
+__device__ __forceinline__ void gs_load_state(f32x2 (&S)[KI / 2][CW], const float* st, int col0, int C, int D, int lane) {
 #pragma unroll
-    for (int c = 0; c < GS_CW; ++c)
+    for (int c = 0; c < CW; ++c)
 #pragma unroll
         for (int p = 0; p < KI / 2; p += (KI == 2 ? 1 : 2)) {
             const int d = gs_channel<KI>(lane, p);
@@ -138,10 +138,10 @@ __device__ __forceinline__ void gs_load_state(f32x2 (&S)[KI / 2][GS_CW], const f
             }
         }
 }
-template <int KI>
-__device__ __forceinline__ void gs_store_state(const f32x2 (&S)[KI / 2][GS_CW], float* st, int col0, int C, int D, int lane) {
+template <int KI, int CW>
+__device__ __forceinline__ void gs_store_state(const f32x2 (&S)[KI / 2][CW], float* st, int col0, int C, int D, int lane) {
 #pragma unroll
-    for (int c = 0; c < GS_CW; ++c)
+    for (int c = 0; c < CW; ++c)
 #pragma unroll
         for (int p = 0; p < KI / 2; p += (KI == 2 ? 1 : 2)) {
             const int d = gs_channel<KI>(lane, p);
@@ -181,13 +181,14 @@ struct GatedScanArgs {
 
 // ----------------------------------------------------------------------------------------
 // Scan over many tokens.  A block takes one sequence, one head and GS_COLS columns of S (columns do not depend on one
-// another); a warp keeps GS_CW columns with all their channels spread over its lanes in registers.  The inputs of TB tokens
-// at a time are copied into a ring of GS_STAGES stages of shared memory by cp.async.  GS_U tokens are worked on side by
-// side: only S is carried from one to the next (one fused multiply-add per value), and their results are summed over the
+// another); a warp keeps CW columns with all their channels spread over its lanes in registers (two columns per warp
+// and twice the warps read shared memory twice as often and were slower at every size).  A warp of its own copies the inputs,
+// TB tokens at a time, into a ring of GS_STAGES stages of shared memory by cp.async.  GS_U tokens are worked on side by side: only S is carried from one to the next (one fused multiply-add per value), and their results are summed over the
 // lanes together, each lane ending up with one (token, column).
 // ----------------------------------------------------------------------------------------
 template <int KI, bool HEAD_GATES>
-__global__ void __launch_bounds__(GS_WARPS * 32) gated_scan_kernel(GatedScanArgs a, int vec) {
+__global__ void __launch_bounds__(GS_THREADS + 32) gated_scan_kernel(GatedScanArgs a, int vec) {
+    constexpr int CW = GS_CW, WARPS = GS_COLS / CW, THREADS = GS_THREADS + 32;       // the working warps, and the one that copies
     constexpr int NB = 32 * KI;
     constexpr int TB = KI >= 8 ? 8 : 16;
     constexpr int ARR = HEAD_GATES ? 2 : 3;
@@ -195,69 +196,86 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gated_scan_kernel(GatedScanArgs
     extern __shared__ __align__(16) float gs_smem[];
     pdl_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int seq = blockIdx.x, head = blockIdx.y, j0 = blockIdx.z * GS_COLS, col0 = j0 + warp * GS_CW;
+    const int seq = blockIdx.x, head = blockIdx.y, j0 = blockIdx.z * GS_COLS, col0 = j0 + warp * CW;
     const int D = a.D;
     // channels past the head's last stay zero in every stage: the copies never touch them
-    for (int i = tid; i < GS_STAGES * STAGE; i += GS_WARPS * 32) gs_smem[i] = 0.f;
+    for (int i = tid; i < GS_STAGES * STAGE; i += THREADS) gs_smem[i] = 0.f;
     pdl_wait();
     const int slot = a.seq_slot[seq];
     const int row0 = a.seq_first_row[seq], n_tok = a.seq_first_row[seq + 1] - row0;
     if (slot < 0 || n_tok <= 0) return;
     float* st = a.state + (int64_t)slot * a.state_stride + (int64_t)head * a.C * D;
-    f32x2 S[KI / 2][GS_CW];
-    gs_load_state<KI>(S, st, col0, a.C, D, lane);
+    const int n_stages = (n_tok + TB - 1) / TB;
     __syncthreads();
 
-    const int n_stages = (n_tok + TB - 1) / TB;
-    auto fetch = [&](int stage) {
-        if (stage < n_stages) {
-            float* base = gs_smem + (stage % GS_STAGES) * STAGE;
-            const int t0 = stage * TB;
-#pragma unroll
-            for (int x = 0; x < TB / GS_WARPS; ++x) {
-                const int t = warp + x * GS_WARPS;
-                if (t0 + t >= n_tok) break;
-                const int64_t row = row0 + t0 + t;
-                const float* src[3] = {a.q + row * a.q_ld + (int64_t)head * D, a.k + row * a.k_ld + (int64_t)head * D,
-                                       HEAD_GATES ? nullptr : a.w + row * a.w_ld + (int64_t)head * D};
+    if (warp == WARPS) {
+        const int64_t hd0 = (int64_t)head * D, hv0 = (int64_t)head * a.V + j0;
+        const float* src[3] = {a.q + row0 * a.q_ld + hd0, a.k + row0 * a.k_ld + hd0, HEAD_GATES ? nullptr : a.w + row0 * a.w_ld + hd0};
+        const int64_t ld[3] = {a.q_ld, a.k_ld, a.w_ld};
+        auto fetch = [&](int stage) {
+            if (stage < n_stages) {
+                float* base = gs_smem + (stage % GS_STAGES) * STAGE;
+                const int t0 = stage * TB, nt = min(TB, n_tok - t0);
 #pragma unroll
                 for (int r = 0; r < ARR; ++r) {
-                    float* dst = base + (r * TB + t) * NB;
+                    const float* p = src[r] + t0 * ld[r];
+                    float* dst = base + r * TB * NB;
                     if (vec) {
+#pragma unroll 4
+                        for (int t = 0; t < nt; ++t, p += ld[r], dst += NB)
 #pragma unroll
-                        for (int c = 4 * lane; c < NB; c += 128)
-                            if (c < D) gs_cp16(dst + c, src[r] + c);
+                            for (int c = 4 * lane; c < NB; c += 128)
+                                if (c < D) gs_cp16(dst + c, p + c);
                     } else {
-                        for (int c = lane; c < D; c += 32) gs_cp4(dst + c, src[r] + c, true);
+                        for (int t = 0; t < nt; ++t, p += ld[r], dst += NB)
+                            for (int c = lane; c < D; c += 32) gs_cp4(dst + c, p + c, true);
                     }
                 }
-            }
-            float* vb = base + ARR * TB * NB;
+                float* vb = base + ARR * TB * NB;
+                const float* pv = a.v + (row0 + t0) * a.v_ld + hv0;
 #pragma unroll
-            for (int x = 0; x < TB * GS_COLS / (GS_WARPS * 32); ++x) {
-                const int e = tid + x * GS_WARPS * 32, t = e / GS_COLS, c = e % GS_COLS;
-                const bool ok = t0 + t < n_tok && j0 + c < a.V;
-                gs_cp4(vb + t * GS_COLS + c, ok ? a.v + (int64_t)(row0 + t0 + t) * a.v_ld + (int64_t)head * a.V + j0 + c : a.v, ok);
+                for (int x = 0; x < TB * GS_COLS / 32; ++x) {
+                    const int e = lane + x * 32, t = e / GS_COLS, c = e % GS_COLS;
+                    const bool ok = t < nt && j0 + c < a.V;
+                    gs_cp4(vb + e, ok ? pv + t * a.v_ld + c : a.v, ok);
+                }
+                if (HEAD_GATES && lane < 2 * TB) {
+                    const int t = lane >> 1;
+                    const bool ok = t < nt;
+                    gs_cp4(vb + TB * GS_COLS + lane, ok ? a.gates + ((int64_t)(row0 + t0 + t) * a.heads + head) * 2 + (lane & 1) : a.gates, ok);
+                }
             }
-            if (HEAD_GATES && tid < 2 * TB) {
-                const int t = tid >> 1;
-                const bool ok = t0 + t < n_tok;
-                gs_cp4(vb + TB * GS_COLS + tid, ok ? a.gates + ((int64_t)(row0 + t0 + t) * a.heads + head) * 2 + (tid & 1) : a.gates, ok);
-            }
+            asm volatile("cp.async.commit_group;" ::: "memory");
+        };
+#pragma unroll
+        for (int s = 0; s < GS_STAGES - 1; ++s) fetch(s);
+        for (int s = 0; s < n_stages; ++s) {
+            asm volatile("cp.async.wait_group %0;" ::"n"(GS_STAGES - 2) : "memory");
+            __syncthreads();                // stage s has arrived, and the working warps are done with stage s - 1
+            fetch(s + GS_STAGES - 1);
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        return;
+    }
+
+    f32x2 S[KI / 2][CW];
+    gs_load_state<KI, CW>(S, st, col0, a.C, D, lane);
     auto token = [&](const float* base, int t, float* acc) {
-        f32x2 q[KI / 2], k[KI / 2], w[KI / 2], v[GS_CW];
+        f32x2 q[KI / 2], k[KI / 2], w[KI / 2], v[CW];
         gs_load_pairs<KI>(q, base + t * NB, lane);
         gs_load_pairs<KI>(k, base + (TB + t) * NB, lane);
         const float* vb = base + ARR * TB * NB;
-        const float4 v4 = *reinterpret_cast<const float4*>(vb + t * GS_COLS + warp * GS_CW);
-        float vv[4] = {v4.x, v4.y, v4.z, v4.w};
+        float vv[CW];
+#pragma unroll
+        for (int c = 0; c < CW; c += 2) {
+            const float2 x = *reinterpret_cast<const float2*>(vb + t * GS_COLS + warp * CW + c);
+            vv[c] = x.x;
+            vv[c + 1] = x.y;
+        }
         if (HEAD_GATES) {
             const float2 g = *reinterpret_cast<const float2*>(vb + TB * GS_COLS + 2 * t);
 #pragma unroll
-            for (int c = 0; c < GS_CW; ++c) {
+            for (int c = 0; c < CW; ++c) {
                 if (col0 + c == a.V) vv[c] = 1.0f;          // the key sum's column
                 vv[c] *= g.y;
             }
@@ -268,8 +286,8 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gated_scan_kernel(GatedScanArgs
             gs_load_pairs<KI>(w, base + (2 * TB + t) * NB, lane);
         }
 #pragma unroll
-        for (int c = 0; c < GS_CW; ++c) v[c] = gs_dup(vv[c]);
-        gs_step<KI>(S, q, k, w, v, acc);
+        for (int c = 0; c < CW; ++c) v[c] = gs_dup(vv[c]);
+        gs_step<KI, CW>(S, q, k, w, v, acc);
     };
     auto put = [&](int t, int c, float x) {
         const int64_t row = row0 + t;
@@ -277,34 +295,36 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gated_scan_kernel(GatedScanArgs
         else if (HEAD_GATES && col0 + c == a.V) a.nq[row * a.heads + head] = x;
     };
 
-#pragma unroll
-    for (int s = 0; s < GS_STAGES - 1; ++s) fetch(s);
+    // after a group of tokens this lane holds the result of token grp_t of the group in column grp_col
+    constexpr int SHARE = 32 / (GS_U * CW);
+    const int grp_t = lane / SHARE / CW, grp_col = col0 + lane / SHARE % CW;
+    const bool grp_sum = HEAD_GATES && grp_col == a.V, grp_live = lane % SHARE == 0 && grp_col < a.C;
+    const int64_t grp_ld = grp_sum ? a.heads : (int64_t)a.heads * a.V;
+    float* grp_dst = (grp_sum ? a.nq + head : a.o + (int64_t)head * a.V + grp_col) + (row0 + grp_t) * grp_ld;
+
     for (int s = 0; s < n_stages; ++s) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(GS_STAGES - 2) : "memory");
-        __syncthreads();                    // stage s has arrived for every thread, and stage s - 1 is done with
-        fetch(s + GS_STAGES - 1);
+        __syncthreads();
         const float* base = gs_smem + (s % GS_STAGES) * STAGE;
         const int t0 = s * TB, nt = min(TB, n_tok - t0);
         if (col0 >= a.C) continue;
         int t = 0;
 #pragma unroll 1
         for (; t + GS_U <= nt; t += GS_U) {
-            float acc[GS_U * GS_CW];
+            float acc[GS_U * CW];
 #pragma unroll
-            for (int u = 0; u < GS_U; ++u) token(base, t + u, acc + u * GS_CW);
-            const float x = gs_reduce<GS_U * GS_CW>(acc, lane);
-            if ((lane & 1) == 0) put(t0 + t + (lane >> 3), (lane >> 1) & 3, x);
+            for (int u = 0; u < GS_U; ++u) token(base, t + u, acc + u * CW);
+            const float x = gs_reduce<GS_U * CW>(acc, lane);
+            if (grp_live) grp_dst[(t0 + t) * grp_ld] = x;
         }
 #pragma unroll 1
         for (; t < nt; ++t) {
-            float acc[GS_CW];
+            float acc[CW];
             token(base, t, acc);
-            const float x = gs_reduce<GS_CW>(acc, lane);
-            if ((lane & 7) == 0) put(t0 + t, lane >> 3, x);
+            const float x = gs_reduce<CW>(acc, lane);
+            if (lane % (32 / CW) == 0) put(t0 + t, lane / (32 / CW), x);
         }
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    gs_store_state<KI>(S, st, col0, a.C, D, lane);
+    gs_store_state<KI, CW>(S, st, col0, a.C, D, lane);
 }
 
 // Any D: S stays in global memory; a thread owns a column.
@@ -368,80 +388,80 @@ __device__ __forceinline__ void gs_head_gate(float i, float f, float& m, float& 
 }
 
 template <int KI, bool HEAD_GATES>
-__global__ void __launch_bounds__(GS_WARPS * 32) gated_step_kernel(GatedScanArgs a, GatedRaw x) {
+__global__ void __launch_bounds__(GS_THREADS) gated_step_kernel(GatedScanArgs a, GatedRaw x) {
     pdl_launch_dependents();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * GS_COLS + warp * GS_CW;
+    // the block's threads work the gates out once, a channel each, and leave them where every column's lanes read them
+    constexpr int CW = GS_CW, NB = 32 * KI, PER = (NB + GS_THREADS - 1) / GS_THREADS;
+    __shared__ __align__(16) float qs[NB], ks[NB], ws[HEAD_GATES ? 4 : NB];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * GS_COLS + warp * CW;
     const int D = a.D;
-    float low[KI], fb[KI];
+    float low[PER], fb[PER];
+    if (!HEAD_GATES) {
 #pragma unroll
-    for (int e = 0; e < KI; ++e) {
-        const int d = gs_channel<KI>(lane, e >> 1) + (e & 1);
-        low[e] = !HEAD_GATES && d < D ? x.lower[(int64_t)head * D + d] : 0.f;
-        fb[e] = !HEAD_GATES && d < D ? x.f_bias[(int64_t)head * D + d] : 0.f;
+        for (int e = 0; e < PER; ++e) {
+            const int d = tid + e * GS_THREADS;
+            low[e] = d < D ? x.lower[(int64_t)head * D + d] : 0.f;
+            fb[e] = d < D ? x.f_bias[(int64_t)head * D + d] : 0.f;
+        }
     }
     const float hfb = HEAD_GATES ? x.f_bias[head] : 0.f, hib = HEAD_GATES ? x.i_bias[head] : 0.f;
     pdl_wait();
     const int slot = a.seq_slot[seq];
     const int row0 = a.seq_first_row[seq], n_tok = a.seq_first_row[seq + 1] - row0;
-    if (slot < 0 || n_tok != 1 || col0 >= a.C) return;
+    if (slot < 0 || n_tok != 1) return;
     float* st = a.state + (int64_t)slot * a.state_stride + (int64_t)head * a.C * D;
-    f32x2 S[KI / 2][GS_CW];
-    gs_load_state<KI>(S, st, col0, a.C, D, lane);
+    f32x2 S[KI / 2][CW];
+    gs_load_state<KI, CW>(S, st, col0, a.C, D, lane);
     const float* row = x.src + (int64_t)row0 * x.ld;
-    float qs[KI], ks[KI], ws[KI], vv[GS_CW];
+    float vv[CW];
 #pragma unroll
-    for (int e = 0; e < KI; ++e) {
-        const int d = gs_channel<KI>(lane, e >> 1) + (e & 1);
-        qs[e] = d < D ? row[x.q_col + (int64_t)head * D + d] : 0.f;
-        ks[e] = d < D ? row[x.k_col + (int64_t)head * D + d] : 0.f;
-        ws[e] = 0.f;
+    for (int c = 0; c < CW; ++c) vv[c] = col0 + c < a.V ? row[x.v_col + (int64_t)head * a.V + col0 + c] : 0.f;
+#pragma unroll
+    for (int e = 0; e < PER; ++e) {
+        const int d = tid + e * GS_THREADS;
+        if (d >= NB) break;
+        float q = 0.f, k = 0.f, f = 0.f;
+        if (d < D) {
+            q = row[x.q_col + (int64_t)head * D + d];
+            k = row[x.k_col + (int64_t)head * D + d];
+            if (!HEAD_GATES) {
+                q = gs_silu(q);
+                gs_channel_gate(k + fb[e], low[e], k, f);
+            }
+        }
+        qs[d] = q;
+        ks[d] = k;
+        if (!HEAD_GATES) ws[d] = f;
     }
-#pragma unroll
-    for (int c = 0; c < GS_CW; ++c) vv[c] = col0 + c < a.V ? row[x.v_col + (int64_t)head * a.V + col0 + c] : 0.f;
+    f32x2 q[KI / 2], k[KI / 2], w[KI / 2], v[CW];
     if (HEAD_GATES) {
         float* mm = a.state + (int64_t)slot * a.state_stride + x.m_off + 2 * head;
         const int pos = x.seq_pos0[seq];
         float m = mm[(pos + 1) & 1], decay, write;
         gs_head_gate(gs_capped(row[x.i_col + head] + hib, x.cap), gs_log_sigmoid(gs_capped(row[x.f_col + head] + hfb, x.cap)), m, decay, write);
-        if (blockIdx.z == 0 && threadIdx.x == 0) {
+        if (blockIdx.z == 0 && tid == 0) {
             mm[pos & 1] = m;
             x.em[(int64_t)row0 * a.heads + head] = expf(-m);
         }
 #pragma unroll
-        for (int e = 0; e < KI; ++e) ws[e] = decay;
+        for (int c = 0; c < CW; ++c) vv[c] = (col0 + c == a.V ? 1.0f : vv[c]) * write;
 #pragma unroll
-        for (int c = 0; c < GS_CW; ++c) {
-            if (col0 + c == a.V) vv[c] = 1.0f;
-            vv[c] *= write;
-        }
-    } else {
-#pragma unroll
-        for (int e = 0; e < KI; ++e) {
-            const int d = gs_channel<KI>(lane, e >> 1) + (e & 1);
-            qs[e] = gs_silu(qs[e]);
-            float k, f;
-            gs_channel_gate(ks[e] + fb[e], low[e], k, f);
-            ks[e] = d < D ? k : 0.f;
-            ws[e] = d < D ? f : 0.f;
-        }
+        for (int p = 0; p < KI / 2; ++p) w[p] = gs_dup(decay);
     }
-    f32x2 q[KI / 2], k[KI / 2], w[KI / 2], v[GS_CW];
+    __syncthreads();
+    gs_load_pairs<KI>(q, qs, lane);
+    gs_load_pairs<KI>(k, ks, lane);
+    if (!HEAD_GATES) gs_load_pairs<KI>(w, ws, lane);
 #pragma unroll
-    for (int p = 0; p < KI / 2; ++p) {
-        q[p] = gs_pack(qs[2 * p], qs[2 * p + 1]);
-        k[p] = gs_pack(ks[2 * p], ks[2 * p + 1]);
-        w[p] = gs_pack(ws[2 * p], ws[2 * p + 1]);
-    }
-#pragma unroll
-    for (int c = 0; c < GS_CW; ++c) v[c] = gs_dup(vv[c]);
-    float acc[GS_CW];
-    gs_step<KI>(S, q, k, w, v, acc);
-    gs_store_state<KI>(S, st, col0, a.C, D, lane);
-    const float r = gs_reduce<GS_CW>(acc, lane);
-    const int c = lane >> 3;
-    if ((lane & 7) == 0) {
-        if (col0 + c < a.V) a.o[(int64_t)row0 * ((int64_t)a.heads * a.V) + (int64_t)head * a.V + col0 + c] = r;
+    for (int c = 0; c < CW; ++c) v[c] = gs_dup(vv[c]);
+    float acc[CW];
+    gs_step<KI, CW>(S, q, k, w, v, acc);
+    gs_store_state<KI, CW>(S, st, col0, a.C, D, lane);
+    const float r = gs_reduce<CW>(acc, lane);
+    const int c = lane / (32 / CW);
+    if (lane % (32 / CW) == 0) {
+        if (col0 + c < a.V) a.o[(int64_t)row0 * a.heads * a.V + (int64_t)head * a.V + col0 + c] = r;
         else if (HEAD_GATES && col0 + c == a.V) a.nq[(int64_t)row0 * a.heads + head] = r;
     }
 }
@@ -486,47 +506,74 @@ __global__ void channel_gates_vec_kernel(GatedRaw x, float* __restrict__ out, in
     }
 }
 
-// Head gates: a warp per (sequence, head) walks the running maximum token by token; 32 tokens' gates are worked out side by
-// side, one per lane, before and after the walk.
-__global__ void __launch_bounds__(32) head_gates_kernel(GatedRaw x, float* __restrict__ gates, float* __restrict__ state, int64_t state_stride,
-                                                        const int32_t* __restrict__ seq_first_row, const int32_t* __restrict__ seq_slot, int heads) {
-    pdl_prologue();
-    const int lane = threadIdx.x, seq = blockIdx.x, head = blockIdx.y;
+// Head gates: a block per (sequence, head).  All threads work out the gates of GS_GATE_TOKENS tokens, one thread walks the
+// running maximum through them (an addition and a maximum per token), all threads turn that into decays and write strengths.
+#define GS_GATE_TOKENS 1024
+__global__ void __launch_bounds__(256) head_gates_kernel(GatedRaw x, float* __restrict__ gates, float* __restrict__ state, int64_t state_stride,
+                                                         const int32_t* __restrict__ seq_first_row, const int32_t* __restrict__ seq_slot, int heads) {
+    __shared__ __align__(16) float is[GS_GATE_TOKENS + 8], fs[GS_GATE_TOKENS + 8], ms[GS_GATE_TOKENS];     // ms: the maximum before a token
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, seq = blockIdx.x, head = blockIdx.y;
+    const float fb = x.f_bias[head], ib = x.i_bias[head];
+    pdl_wait();
     const int slot = seq_slot[seq];
     const int row0 = seq_first_row[seq], n_tok = seq_first_row[seq + 1] - row0;
     if (slot < 0 || n_tok <= 0) return;
     const int pos0 = x.seq_pos0[seq];
     float* mm = state + (int64_t)slot * state_stride + x.m_off + 2 * head;
-    float m = mm[(pos0 + 1) & 1];
-    const float fb = x.f_bias[head], ib = x.i_bias[head];
-    float i_next = 0.f, f_next = 0.f;
-    auto fetch = [&](int t0) {
-        const int t = min(t0 + lane, n_tok - 1);
-        const float* src = x.src + (int64_t)(row0 + t) * x.ld;
-        i_next = src[x.i_col + head];
-        f_next = src[x.f_col + head];
-    };
-    fetch(0);
-    for (int t0 = 0; t0 < n_tok; t0 += 32) {
-        const float i = gs_capped(i_next + ib, x.cap), f = gs_log_sigmoid(gs_capped(f_next + fb, x.cap));
-        if (t0 + 32 < n_tok) fetch(t0 + 32);
-        const int nt = min(32, n_tok - t0);
-        float before = m;
+    float m = tid == 0 ? mm[(pos0 + 1) & 1] : 0.f;
+    for (int t0 = 0; t0 < n_tok; t0 += GS_GATE_TOKENS) {
+        const int nt = min(GS_GATE_TOKENS, n_tok - t0);
+        const int padded = (nt + 7) / 8 * 8;
+        float ri[GS_GATE_TOKENS / 256], rf[GS_GATE_TOKENS / 256];
 #pragma unroll
-        for (int t = 0; t < 32; ++t) {
-            const float it = __shfl_sync(0xffffffffu, i, t), ft = __shfl_sync(0xffffffffu, f, t);
-            if (t == lane) before = m;
-            if (t < nt) m = fmaxf(ft + m, it);
+        for (int e = 0; e < GS_GATE_TOKENS / 256; ++e) {
+            const float* src = x.src + (int64_t)(row0 + t0 + min(tid + 256 * e, nt - 1)) * x.ld;
+            ri[e] = src[x.i_col + head];
+            rf[e] = src[x.f_col + head];
         }
-        if (lane < nt) {
-            float decay, write;
-            gs_head_gate(i, f, before, decay, write);
-            const int64_t at = (int64_t)(row0 + t0 + lane) * heads + head;
+#pragma unroll
+        for (int e = 0; e < GS_GATE_TOKENS / 256; ++e) {
+            const int t = tid + 256 * e;
+            if (t < padded) {           // (places past the last token leave the maximum as it is)
+                is[t] = t < nt ? gs_capped(ri[e] + ib, x.cap) : -INFINITY;
+                fs[t] = t < nt ? gs_log_sigmoid(gs_capped(rf[e] + fb, x.cap)) : 0.f;
+            }
+        }
+        __syncthreads();
+        if (tid == 0) {
+            // eight tokens at a time, the next eight on their way: a token costs an addition and a maximum, no read to wait for
+            float4 f0 = *reinterpret_cast<float4*>(fs), f1 = *reinterpret_cast<float4*>(fs + 4);
+            float4 i0 = *reinterpret_cast<float4*>(is), i1 = *reinterpret_cast<float4*>(is + 4);
+#pragma unroll 2
+            for (int t = 0; t < padded; t += 8) {
+                const float4 nf0 = *reinterpret_cast<float4*>(fs + t + 8), nf1 = *reinterpret_cast<float4*>(fs + t + 12);
+                const float4 ni0 = *reinterpret_cast<float4*>(is + t + 8), ni1 = *reinterpret_cast<float4*>(is + t + 12);
+                float4 b0, b1;
+                b0.x = m; m = fmaxf(f0.x + m, i0.x);
+                b0.y = m; m = fmaxf(f0.y + m, i0.y);
+                b0.z = m; m = fmaxf(f0.z + m, i0.z);
+                b0.w = m; m = fmaxf(f0.w + m, i0.w);
+                b1.x = m; m = fmaxf(f1.x + m, i1.x);
+                b1.y = m; m = fmaxf(f1.y + m, i1.y);
+                b1.z = m; m = fmaxf(f1.z + m, i1.z);
+                b1.w = m; m = fmaxf(f1.w + m, i1.w);
+                *reinterpret_cast<float4*>(ms + t) = b0;
+                *reinterpret_cast<float4*>(ms + t + 4) = b1;
+                f0 = nf0; f1 = nf1; i0 = ni0; i1 = ni1;
+            }
+        }
+        __syncthreads();
+        for (int t = tid; t < nt; t += 256) {
+            float before = ms[t], decay, write;
+            gs_head_gate(is[t], fs[t], before, decay, write);
+            const int64_t at = (int64_t)(row0 + t0 + t) * heads + head;
             *reinterpret_cast<float2*>(gates + 2 * at) = make_float2(decay, write);
             x.em[at] = expf(-before);
         }
+        __syncthreads();
     }
-    if (lane == 0) mm[(pos0 + n_tok - 1) & 1] = m;
+    if (tid == 0) mm[(pos0 + n_tok - 1) & 1] = m;
 }
 
 // ----------------------------------------------------------------------------------------
@@ -559,7 +606,7 @@ template <> __device__ __forceinline__ void gs_store4<bf16>(bf16* p, float a, fl
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
 }
 
-template <typename T, bool VEC>
+template <typename T>
 __global__ void scan_head_norm_kernel(HeadNormArgs a, T* __restrict__ out, int64_t items) {
     pdl_prologue();
     const int lane = threadIdx.x & 31;
@@ -574,40 +621,51 @@ __global__ void scan_head_norm_kernel(HeadNormArgs a, T* __restrict__ out, int64
     const float* g = a.gate != nullptr ? a.gate + row * a.gate_ld + (int64_t)head * a.V : nullptr;
     T* dst = out + row * a.out_ld + (int64_t)head * a.V;
     float ss = 0.f;
-    if (VEC) {
-        float4 first = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int i = 4 * lane; i < a.V; i += 128) {
-            float4 v = *reinterpret_cast<const float4*>(src + i);
-            v.x *= f; v.y *= f; v.z *= f; v.w *= f;
-            if (i < 128) first = v;
-            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    for (int i = lane; i < a.V; i += 32) {
+        const float v = src[i] * f;
+        ss = fmaf(v, v, ss);
+    }
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)a.V + a.eps) * a.post;
+    for (int i = lane; i < a.V; i += 32) {
+        float y = src[i] * f * r * w[i];
+        if (g != nullptr) y *= gs_sigmoid(g[i]);
+        dst[i] = from_f32<T>(y);
+    }
+}
+
+// The same for V a multiple of 4 up to 128 and 16-byte aligned rows: a lane has 4 values of a head, a warp ITEMS heads at once,
+// all of whose reads are asked for before any is used.
+template <typename T, int ITEMS>
+__global__ void __launch_bounds__(128) scan_head_norm_vec_kernel(HeadNormArgs a, T* __restrict__ out, int64_t items) {
+    pdl_prologue();
+    const int lane = threadIdx.x & 31, i = 4 * lane;
+    const int64_t item0 = ((int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * ITEMS;
+    const bool in = i < a.V;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 v[ITEMS], g[ITEMS], w[ITEMS];
+    float f[ITEMS];
+    int64_t at[ITEMS];
+#pragma unroll
+    for (int x = 0; x < ITEMS; ++x) {
+        const int64_t item = item0 + x < items ? item0 + x : items - 1;
+        const int64_t row = item / a.heads;
+        const int head = (int)(item - row * a.heads);
+        at[x] = row * a.out_ld + (int64_t)head * a.V + i;
+        v[x] = in ? *reinterpret_cast<const float4*>(a.o + item * a.V + i) : zero;
+        w[x] = in ? *reinterpret_cast<const float4*>(a.weight + (a.shared ? 0 : (int64_t)head * a.V) + i) : zero;
+        g[x] = in && a.gate != nullptr ? *reinterpret_cast<const float4*>(a.gate + row * a.gate_ld + (int64_t)head * a.V + i) : zero;
+        f[x] = a.nq != nullptr ? a.q_scale / (fmaxf(fabsf(a.nq[item] * a.q_scale), a.em[item]) + a.tiny) : 1.f;
+    }
+#pragma unroll
+    for (int x = 0; x < ITEMS; ++x) {
+        v[x].x *= f[x]; v[x].y *= f[x]; v[x].z *= f[x]; v[x].w *= f[x];
+        const float ss = warp_sum(fmaf(v[x].x, v[x].x, fmaf(v[x].y, v[x].y, fmaf(v[x].z, v[x].z, v[x].w * v[x].w))));
+        const float r = 1.0f / sqrtf(ss / (float)a.V + a.eps) * a.post;
+        float y[4] = {v[x].x * r * w[x].x, v[x].y * r * w[x].y, v[x].z * r * w[x].z, v[x].w * r * w[x].w};
+        if (a.gate != nullptr) {
+            y[0] *= gs_sigmoid(g[x].x); y[1] *= gs_sigmoid(g[x].y); y[2] *= gs_sigmoid(g[x].z); y[3] *= gs_sigmoid(g[x].w);
         }
-        const float r = 1.0f / sqrtf(warp_sum(ss) / (float)a.V + a.eps) * a.post;
-        for (int i = 4 * lane; i < a.V; i += 128) {
-            float4 v = first;
-            if (i >= 128) {
-                v = *reinterpret_cast<const float4*>(src + i);
-                v.x *= f; v.y *= f; v.z *= f; v.w *= f;
-            }
-            const float4 wv = *reinterpret_cast<const float4*>(w + i);
-            float y[4] = {v.x * r * wv.x, v.y * r * wv.y, v.z * r * wv.z, v.w * r * wv.w};
-            if (g != nullptr) {
-                const float4 gv = *reinterpret_cast<const float4*>(g + i);
-                y[0] *= gs_sigmoid(gv.x); y[1] *= gs_sigmoid(gv.y); y[2] *= gs_sigmoid(gv.z); y[3] *= gs_sigmoid(gv.w);
-            }
-            gs_store4<T>(dst + i, y[0], y[1], y[2], y[3]);
-        }
-    } else {
-        for (int i = lane; i < a.V; i += 32) {
-            const float v = src[i] * f;
-            ss = fmaf(v, v, ss);
-        }
-        const float r = 1.0f / sqrtf(warp_sum(ss) / (float)a.V + a.eps) * a.post;
-        for (int i = lane; i < a.V; i += 32) {
-            float y = src[i] * f * r * w[i];
-            if (g != nullptr) y *= gs_sigmoid(g[i]);
-            dst[i] = from_f32<T>(y);
-        }
+        if (in && item0 + x < items) gs_store4<T>(out + at[x], y[0], y[1], y[2], y[3]);
     }
 }
 
@@ -626,7 +684,9 @@ static int gated_scan_launch(const GatedScanArgs& a, int n_seqs, int vec, cudaSt
         X0NE_REQUIRE(e == cudaSuccess, "gated_scan: %zu bytes of shared memory: %s", SMEM, cudaGetErrorString(e));
         configured.done();
     }
-    x0ne_launch(gated_scan_kernel<KI, HEAD_GATES>, dim3(n_seqs, a.heads, (a.C + GS_COLS - 1) / GS_COLS), dim3(GS_WARPS * 32), SMEM, stream, a, vec);
+    // Launched without the early-start attribute: blocks that start while the kernel before still fills the GPU gather on the
+    // first multiprocessors that have room, two on one while others stay empty, and stay there for the whole scan.
+    gated_scan_kernel<KI, HEAD_GATES><<<dim3(n_seqs, a.heads, (a.C + GS_COLS - 1) / GS_COLS), dim3(GS_THREADS + 32), SMEM, stream>>>(a, vec);
     X0NE_LAUNCH_CHECK();
 }
 
@@ -652,9 +712,11 @@ X0NE_API int x0ne_gated_scan(GatedScanArgs a, int n_seqs, cudaStream_t stream) {
         x0ne_launch(gated_scan_any_kernel, dim3(n_seqs, a.heads, (a.C + threads - 1) / threads), dim3(threads), 0, stream, a);
         X0NE_LAUNCH_CHECK();
     }
-    if (a.D <= 64) return hg ? gated_scan_launch<2, true>(a, n_seqs, vec, stream) : gated_scan_launch<2, false>(a, n_seqs, vec, stream);
-    if (a.D <= 128) return hg ? gated_scan_launch<4, true>(a, n_seqs, vec, stream) : gated_scan_launch<4, false>(a, n_seqs, vec, stream);
-    return hg ? gated_scan_launch<8, true>(a, n_seqs, vec, stream) : gated_scan_launch<8, false>(a, n_seqs, vec, stream);
+#define GS_SCAN(KI) return hg ? gated_scan_launch<KI, true>(a, n_seqs, vec, stream) : gated_scan_launch<KI, false>(a, n_seqs, vec, stream)
+    if (a.D <= 64) GS_SCAN(2);
+    if (a.D <= 128) GS_SCAN(4);
+    GS_SCAN(8);
+#undef GS_SCAN
 }
 
 // The widest head whose one-token steps x0ne_gated_step takes (wider ones go through the gates' kernels and the scan).
@@ -668,7 +730,7 @@ X0NE_API int x0ne_gated_step(GatedScanArgs a, GatedRaw x, int n_seqs, cudaStream
     X0NE_REQUIRE(x.src != nullptr && x.f_bias != nullptr && (hg ? x.i_bias != nullptr && x.em != nullptr && x.cap > 0.f && x.seq_pos0 != nullptr &&
                  x.m_off >= (int64_t)a.heads * a.C * a.D && a.state_stride >= x.m_off + 2 * a.heads : x.lower != nullptr), "gated_step: a gate's tensor is missing");
     if (n_seqs == 0) return 0;
-    const dim3 grid(n_seqs, a.heads, (a.C + GS_COLS - 1) / GS_COLS), block(GS_WARPS * 32);
+    const dim3 grid(n_seqs, a.heads, (a.C + GS_COLS - 1) / GS_COLS), block(GS_THREADS);
 #define GS_STEP(KI)                                                                                      \
     do {                                                                                                 \
         if (hg) x0ne_launch(gated_step_kernel<KI, true>, grid, block, 0, stream, a, x);                  \
@@ -699,7 +761,7 @@ X0NE_API int x0ne_head_gates(GatedRaw x, float* gates, float* state, int64_t sta
     X0NE_REQUIRE(n_seqs >= 0 && heads > 0 && heads <= 65535 && x.src != nullptr && x.f_bias != nullptr && x.i_bias != nullptr && x.em != nullptr && x.cap > 0.f &&
                      x.seq_pos0 != nullptr && state_stride >= x.m_off + 2 * heads, "head_gates: %d sequences, %d heads", n_seqs, heads);
     if (n_seqs == 0) return 0;
-    x0ne_launch(head_gates_kernel, dim3(n_seqs, heads), dim3(32), 0, stream, x, gates, state, state_stride, seq_first_row, seq_slot, heads);
+    x0ne_launch(head_gates_kernel, dim3(n_seqs, heads), dim3(256), 0, stream, x, gates, state, state_stride, seq_first_row, seq_slot, heads);
     X0NE_LAUNCH_CHECK();
 }
 
@@ -709,15 +771,19 @@ X0NE_API int x0ne_scan_head_norm(HeadNormArgs a, void* out, int dt, int n_rows, 
     X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "scan_head_norm: unknown dtype tag %d", dt);
     if (n_rows == 0) return 0;
     const int64_t items = (int64_t)n_rows * a.heads;
-    const dim3 grid((unsigned)((items + 3) / 4)), block(128);
-    const bool vec = a.V % 4 == 0 && a.out_ld % 4 == 0 && a.gate_ld % 4 == 0 && gs_aligned16(a.o) && gs_aligned16(a.weight) && gs_aligned16(a.gate) &&
-                     (((uintptr_t)out) & (dt == X0NE_F32 ? 15 : 7)) == 0;
-    if (dt == X0NE_F32) {
-        if (vec) x0ne_launch(scan_head_norm_kernel<float, true>, grid, block, 0, stream, a, (float*)out, items);
-        else x0ne_launch(scan_head_norm_kernel<float, false>, grid, block, 0, stream, a, (float*)out, items);
-    } else {
-        if (vec) x0ne_launch(scan_head_norm_kernel<bf16, true>, grid, block, 0, stream, a, (bf16*)out, items);
-        else x0ne_launch(scan_head_norm_kernel<bf16, false>, grid, block, 0, stream, a, (bf16*)out, items);
-    }
+    const bool vec = a.V % 4 == 0 && a.V <= 128 && a.out_ld % 4 == 0 && a.gate_ld % 4 == 0 && gs_aligned16(a.o) && gs_aligned16(a.weight) &&
+                     gs_aligned16(a.gate) && (((uintptr_t)out) & (dt == X0NE_F32 ? 15 : 7)) == 0;
+    // (a head's sum runs over the same lanes in the same order however many heads a warp has)
+    const int per_warp = vec && items >= 4096 ? 4 : 1;
+    const dim3 grid((unsigned)((items + 4 * per_warp - 1) / (4 * per_warp))), block(128);
+#define GS_HEAD_NORM(T)                                                                                                  \
+    do {                                                                                                                 \
+        if (!vec) x0ne_launch(scan_head_norm_kernel<T>, grid, block, 0, stream, a, (T*)out, items);                      \
+        else if (per_warp == 4) x0ne_launch(scan_head_norm_vec_kernel<T, 4>, grid, block, 0, stream, a, (T*)out, items); \
+        else x0ne_launch(scan_head_norm_vec_kernel<T, 1>, grid, block, 0, stream, a, (T*)out, items);                    \
+    } while (0)
+    if (dt == X0NE_F32) GS_HEAD_NORM(float);
+    else GS_HEAD_NORM(bf16);
+#undef GS_HEAD_NORM
     X0NE_LAUNCH_CHECK();
 }

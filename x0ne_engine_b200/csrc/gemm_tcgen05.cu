@@ -34,7 +34,29 @@ struct TcShared {
     uint64_t accum_empty[2];
     uint32_t tmem_base;
     int failed;
+    __align__(16) float bias[4][256];       // per epilogue warp: a tile's gate biases, then its up biases
 };
+
+// A gated tile's biases into the epilogue warp's own copy (they are the same for every row): asked for before the warp waits
+// for the accumulator, read back 16 bytes at a time.
+__device__ __forceinline__ void tc_stage_bias(float* dst, const float* bias, int n0, int N, int lane) {
+    __syncwarp();               // (the tile before may still be reading)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int n = n0 + 32 * i + lane;
+        dst[32 * i + lane] = n < N ? bias[n] : 0.f;
+        dst[128 + 32 * i + lane] = n < N ? bias[N + n] : 0.f;
+    }
+    __syncwarp();
+}
+__device__ __forceinline__ void tc_add_bias(float (&v)[32], float (&u)[32], const float* bias) {
+#pragma unroll
+    for (int i = 0; i < 32; i += 4) {
+        const float4 g = *reinterpret_cast<const float4*>(bias + i), w = *reinterpret_cast<const float4*>(bias + 128 + i);
+        v[i] += g.x; v[i + 1] += g.y; v[i + 2] += g.z; v[i + 3] += g.w;
+        u[i] += w.x; u[i + 1] += w.y; u[i + 2] += w.z; u[i + 3] += w.w;
+    }
+}
 
 // SWIGLU: W is the packed [gate; up] weight of 2 * N rows; a tile's W operand is gate rows
 // n0 .. n0 + 127 and up rows N + n0 .. N + n0 + 127, and y has N columns.
@@ -153,6 +175,7 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_kernel(const __grid_consta
             const int ab = t & 1;
             const int m0 = (tile % m_tiles) * TC_BM, n0 = (tile / m_tiles) * BN;
             const int m = m0 + quarter * 32 + lane;
+            if (SWIGLU && glu.bias != nullptr) tc_stage_bias(sh->bias[quarter], glu.bias, n0, N, lane);
             if (!mbar_wait(&sh->accum_full[ab], (t >> 1) & 1, status, 3) || sh->failed) {
                 sh->failed = 1;
                 break;
@@ -166,8 +189,9 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_kernel(const __grid_consta
                 if (SWIGLU) {
                     float u[32];
                     tc_ld32(trow + 128 + c * 32, u);
+                    if (glu.bias != nullptr) tc_add_bias(v, u, &sh->bias[quarter][c * 32]);
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = glu_act_at(v[i], u[i], n0 + c * 32 + i, N, glu);
+                    for (int i = 0; i < 32; ++i) v[i] = glu_act(v[i], u[i], glu);
                 }
                 const int n = n0 + c * 32;
                 if (m < M) {
@@ -216,6 +240,7 @@ struct Tc2Shared {
     uint64_t accum_empty[2];
     uint32_t tmem_base;
     int failed;
+    __align__(16) float bias[4][256];       // as in TcShared
 };
 
 __device__ __forceinline__ uint32_t cluster_rank() {
@@ -353,6 +378,7 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_pair_kernel(const __grid_c
             const int ab = t & 1;
             const int m0 = (tile % m_tiles) * 256 + 128 * (int)rank, n0 = (tile / m_tiles) * BN;
             const int m = m0 + quarter * 32 + lane;
+            if (SWIGLU && glu.bias != nullptr) tc_stage_bias(sh->bias[quarter], glu.bias, n0, N, lane);
             if (!mbar_wait(&sh->accum_full[ab], (t >> 1) & 1, status, 3) || sh->failed) {
                 sh->failed = 1;
                 break;
@@ -366,8 +392,9 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_pair_kernel(const __grid_c
                 if (SWIGLU) {
                     float u[32];
                     tc_ld32(trow + 128 + c * 32, u);
+                    if (glu.bias != nullptr) tc_add_bias(v, u, &sh->bias[quarter][c * 32]);
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = glu_act_at(v[i], u[i], n0 + c * 32 + i, N, glu);
+                    for (int i = 0; i < 32; ++i) v[i] = glu_act(v[i], u[i], glu);
                 }
                 const int n = n0 + c * 32;
                 if (m < M) {

@@ -11,6 +11,7 @@
 #include "common.cuh"
 
 #define IC_ROWS 16          // rows of a stretch (at least the taps - 1 whose first rows read the kept inputs)
+#define IC_VEC_ROWS 8       // the same for the vectorised kernel, which takes up to 5 taps
 #define IC_MAX_TAPS 17
 
 __device__ __forceinline__ void ic_load8(const float* p, float* v) {
@@ -38,6 +39,30 @@ __device__ __forceinline__ void ic_store8(bf16* p, const float* v) {
     for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
     *reinterpret_cast<uint4*>(p) = r;
 }
+
+// 8 values as they were read: an instruction that unpacked them would wait for the read
+template <typename T> struct IcRaw;
+template <> struct IcRaw<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) {
+        a = reinterpret_cast<const float4*>(p)[0];
+        b = reinterpret_cast<const float4*>(p)[1];
+    }
+    __device__ __forceinline__ void unpack(float* v) const { v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w; }
+};
+template <> struct IcRaw<bf16> {
+    uint4 a;
+    __device__ __forceinline__ void load(const bf16* p) { a = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void unpack(float* v) const {
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&a);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 f = __bfloat1622float2(h[i]);
+            v[2 * i] = f.x;
+            v[2 * i + 1] = f.y;
+        }
+    }
+};
 
 // Any width and number of taps: a thread per channel; every input is read where it lies.
 template <typename T>
@@ -67,7 +92,7 @@ __global__ void input_conv_any_kernel(const T* __restrict__ h, const float* __re
         }
 }
 
-// TAPS at compile time, 8 channels per thread, the last TAPS - 1 inputs in registers.
+// TAPS at compile time, 8 channels per thread; a stretch's rows are all asked for before the first is used.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) input_conv_vec_kernel(const T* __restrict__ h, const float* __restrict__ w, float* __restrict__ state,
                                                              int64_t state_stride, int64_t off, T* __restrict__ out,
@@ -83,10 +108,14 @@ __global__ void __launch_bounds__(128) input_conv_vec_kernel(const T* __restrict
     }
     pdl_wait();
     const int row0 = seq_first_row[seq], n_tok = seq_first_row[seq + 1] - row0, slot = seq_slot[seq];
-    const int t0 = blockIdx.z * IC_ROWS, t1 = min(n_tok, t0 + IC_ROWS);
+    const int t0 = blockIdx.z * IC_VEC_ROWS, t1 = min(n_tok, t0 + IC_VEC_ROWS);
     if (c >= width || t0 >= n_tok || slot < 0) return;
     float* st = state + (int64_t)slot * state_stride + off + c;
     const T* src = h + (int64_t)row0 * width + c;
+    IcRaw<T> raw[IC_VEC_ROWS];
+#pragma unroll
+    for (int r = 0; r < IC_VEC_ROWS; ++r)
+        if (t0 + r < t1) raw[r].load(src + (int64_t)(t0 + r) * width);
     float win[TAPS][8];                     // the inputs ahead of the row, oldest first, then the row's own
 #pragma unroll
     for (int i = 0; i < KEPT; ++i) {
@@ -94,9 +123,10 @@ __global__ void __launch_bounds__(128) input_conv_vec_kernel(const T* __restrict
         if (at >= 0) ic_load8(src + (int64_t)at * width, win[i]);
         else ic_load8(st + (int64_t)(at + KEPT) * width, win[i]);
     }
-#pragma unroll 4
-    for (int t = t0; t < t1; ++t) {
-        ic_load8(src + (int64_t)t * width, win[KEPT]);
+#pragma unroll
+    for (int r = 0; r < IC_VEC_ROWS; ++r) {
+        if (t0 + r >= t1) break;
+        raw[r].unpack(win[KEPT]);
         float y[8];
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
@@ -105,7 +135,7 @@ __global__ void __launch_bounds__(128) input_conv_vec_kernel(const T* __restrict
             for (int j = 0; j < TAPS; ++j) acc = fmaf(wk[j][e], win[j][e], acc);
             y[e] = win[KEPT][e] + acc;
         }
-        ic_store8(out + (int64_t)(row0 + t) * width + c, y);
+        ic_store8(out + (int64_t)(row0 + t0 + r) * width + c, y);
 #pragma unroll
         for (int i = 0; i < KEPT; ++i)
 #pragma unroll
@@ -130,18 +160,18 @@ X0NE_API int x0ne_input_conv_max_taps() { return IC_MAX_TAPS; }
 X0NE_API int x0ne_input_conv(const void* h, int dt, const float* w, float* state, int64_t state_stride, int64_t off, void* out,
                              const int32_t* seq_first_row, const int32_t* seq_slot, int n_seqs, int max_seq_rows, int width, int taps,
                              cudaStream_t stream) {
-    X0NE_REQUIRE(n_seqs >= 0 && n_seqs <= 65535 && width > 0 && taps >= 1 && taps <= IC_MAX_TAPS && max_seq_rows >= 0 && max_seq_rows <= 65535 * IC_ROWS,
+    X0NE_REQUIRE(n_seqs >= 0 && n_seqs <= 65535 && width > 0 && taps >= 1 && taps <= IC_MAX_TAPS && max_seq_rows >= 0 && max_seq_rows <= 65535 * IC_VEC_ROWS,
                  "input_conv: %d sequences of up to %d rows, width %d, %d taps (at most %d)", n_seqs, max_seq_rows, width, taps, IC_MAX_TAPS);
     X0NE_REQUIRE(taps == 1 || (state != nullptr && off >= 0 && state_stride >= off + (int64_t)(taps - 1) * width), "input_conv: the state row is too short");
     X0NE_REQUIRE(h != out, "input_conv: a row's inputs are read after rows above are written, so it does not run in place");
     X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "input_conv: unknown dtype tag %d", dt);
     if (n_seqs == 0 || max_seq_rows == 0) return 0;
-    const unsigned stretches = (unsigned)((max_seq_rows + IC_ROWS - 1) / IC_ROWS);
     const bool vec = width % 8 == 0 && taps <= 5 && off % 4 == 0 && state_stride % 4 == 0 &&
                      (((uintptr_t)h | (uintptr_t)out | (uintptr_t)w | (uintptr_t)state) & 15) == 0;
     if (vec) {
         const int threads = width / 8 >= 128 ? 128 : (width / 8 + 31) / 32 * 32;
-        const dim3 grid((unsigned)((width / 8 + threads - 1) / threads), (unsigned)n_seqs, stretches), block(threads);
+        const dim3 grid((unsigned)((width / 8 + threads - 1) / threads), (unsigned)n_seqs, (unsigned)((max_seq_rows + IC_VEC_ROWS - 1) / IC_VEC_ROWS)),
+            block(threads);
 #define IC_VEC(K)                                                                                                                        \
         if (dt == X0NE_F32) x0ne_launch(input_conv_vec_kernel<float, K>, grid, block, 0, stream, (const float*)h, w, state, state_stride, off, (float*)out, seq_first_row, seq_slot, width); \
         else x0ne_launch(input_conv_vec_kernel<bf16, K>, grid, block, 0, stream, (const bf16*)h, w, state, state_stride, off, (bf16*)out, seq_first_row, seq_slot, width)
@@ -156,7 +186,7 @@ X0NE_API int x0ne_input_conv(const void* h, int dt, const float* w, float* state
         X0NE_LAUNCH_CHECK();
     }
     const int threads = width >= 128 ? 128 : (width + 31) / 32 * 32;
-    const dim3 grid((unsigned)((width + threads - 1) / threads), (unsigned)n_seqs, stretches);
+    const dim3 grid((unsigned)((width + threads - 1) / threads), (unsigned)n_seqs, (unsigned)((max_seq_rows + IC_ROWS - 1) / IC_ROWS));
     if (dt == X0NE_F32)
         x0ne_launch(input_conv_any_kernel<float>, grid, dim3(threads), 0, stream, (const float*)h, w, state, state_stride, off, (float*)out, seq_first_row, seq_slot, width, taps);
     else

@@ -88,6 +88,9 @@ RULES: List[Rule] = [
     Rule("skinny", (17, 48), False, lambda s: s.weight_bytes >= 64 * MB,
          "10240 x 5120 at 32 rows: skinny 20.1 us, library 21.1; 5120 x 8192: 17.0 / 19.4; at 64 rows the library is ahead on both"),
     # ---- many rows
+    Rule("library", (768, 2048), True, lambda s: s.k <= 2048,
+         "gate|up 12288 x 2048 at 2,048 rows: library 89.8 us with the activation's launch, tc_pair 99.9 (113.1 with biases in the "
+         "epilogue: a tile of 32 steps over K does not cover it)"),
     Rule("tc_pair", (768, 1 << 30), True, _always,
          "gate|up 24576 x 4096 at 2,048 rows: 1.62 PFLOP/s with the activation in the epilogue; at 512 rows the library "
          "(74.9 us + 8.5 for SwiGLU) is ahead of it (84.6)"),
