@@ -597,29 +597,19 @@ struct HeadNormArgs {
     int32_t heads, V;
 };
 
-template <typename T> __device__ __forceinline__ void gs_store4(T* p, float a, float b, float c, float d);
-template <> __device__ __forceinline__ void gs_store4<float>(float* p, float a, float b, float c, float d) {
-    *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
-}
-template <> __device__ __forceinline__ void gs_store4<bf16>(bf16* p, float a, float b, float c, float d) {
-    const __nv_bfloat162 x = __floats2bfloat162_rn(a, b), y = __floats2bfloat162_rn(c, d);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
-}
-
 template <typename T>
-__global__ void scan_head_norm_kernel(HeadNormArgs a, T* __restrict__ out, int64_t items) {
+__global__ void scan_head_norm_kernel(HeadNormArgs a, T* __restrict__ out, uint32_t items) {
     pdl_prologue();
     const int lane = threadIdx.x & 31;
-    const int64_t item = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const uint32_t item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (item >= items) return;
-    const int64_t row = item / a.heads;
-    const int head = (int)(item - row * a.heads);
-    const float* src = a.o + item * a.V;
+    const uint32_t row = item / (uint32_t)a.heads, head = item - row * (uint32_t)a.heads;
+    const float* src = a.o + (int64_t)item * a.V;
     float f = 1.f;
     if (a.nq != nullptr) f = a.q_scale / (fmaxf(fabsf(a.nq[item] * a.q_scale), a.em[item]) + a.tiny);
     const float* w = a.weight + (a.shared ? 0 : (int64_t)head * a.V);
-    const float* g = a.gate != nullptr ? a.gate + row * a.gate_ld + (int64_t)head * a.V : nullptr;
-    T* dst = out + row * a.out_ld + (int64_t)head * a.V;
+    const float* g = a.gate != nullptr ? a.gate + (int64_t)row * a.gate_ld + (int64_t)head * a.V : nullptr;
+    T* dst = out + (int64_t)row * a.out_ld + (int64_t)head * a.V;
     float ss = 0.f;
     for (int i = lane; i < a.V; i += 32) {
         const float v = src[i] * f;
@@ -633,40 +623,52 @@ __global__ void scan_head_norm_kernel(HeadNormArgs a, T* __restrict__ out, int64
     }
 }
 
-// The same for V a multiple of 4 up to 128 and 16-byte aligned rows: a lane has 4 values of a head, a warp ITEMS heads at once,
-// all of whose reads are asked for before any is used.
-template <typename T, int ITEMS>
-__global__ void __launch_bounds__(128) scan_head_norm_vec_kernel(HeadNormArgs a, T* __restrict__ out, int64_t items) {
+// The same for V a multiple of 8 up to 256 and 16-byte aligned rows: LANES lanes (a power of two, the fewest that hold V) have 8
+// values of a head each.
+__device__ __forceinline__ void gs_load8(const float* p, float* v) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void gs_store8(float* p, const float* v) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void gs_store8(bf16* p, const float* v) {
+    uint4 r;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&r);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    *reinterpret_cast<uint4*>(p) = r;
+}
+
+template <typename T, int LANES>
+__global__ void __launch_bounds__(128) scan_head_norm_vec_kernel(HeadNormArgs a, T* __restrict__ out, uint32_t items) {
     pdl_prologue();
-    const int lane = threadIdx.x & 31, i = 4 * lane;
-    const int64_t item0 = ((int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * ITEMS;
-    const bool in = i < a.V;
-    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-    float4 v[ITEMS], g[ITEMS], w[ITEMS];
-    float f[ITEMS];
-    int64_t at[ITEMS];
+    const uint32_t item = (blockIdx.x * 128 + threadIdx.x) / LANES;
+    const int i = (threadIdx.x % LANES) * 8;
+    const bool live = item < items && i < a.V;
+    const uint32_t at = live ? item : 0, row = at / (uint32_t)a.heads, head = at - row * (uint32_t)a.heads;
+    const int c = live ? i : 0;
+    float v[8], g[8], w[8];
+    gs_load8(a.o + (int64_t)at * a.V + c, v);
+    gs_load8(a.weight + (a.shared ? 0 : (int64_t)head * a.V) + c, w);
+    if (a.gate != nullptr) gs_load8(a.gate + (int64_t)row * a.gate_ld + (int64_t)head * a.V + c, g);
+    const float f = a.nq != nullptr ? a.q_scale / (fmaxf(fabsf(a.nq[at] * a.q_scale), a.em[at]) + a.tiny) : 1.f;
+    float ss = 0.f;
 #pragma unroll
-    for (int x = 0; x < ITEMS; ++x) {
-        const int64_t item = item0 + x < items ? item0 + x : items - 1;
-        const int64_t row = item / a.heads;
-        const int head = (int)(item - row * a.heads);
-        at[x] = row * a.out_ld + (int64_t)head * a.V + i;
-        v[x] = in ? *reinterpret_cast<const float4*>(a.o + item * a.V + i) : zero;
-        w[x] = in ? *reinterpret_cast<const float4*>(a.weight + (a.shared ? 0 : (int64_t)head * a.V) + i) : zero;
-        g[x] = in && a.gate != nullptr ? *reinterpret_cast<const float4*>(a.gate + row * a.gate_ld + (int64_t)head * a.V + i) : zero;
-        f[x] = a.nq != nullptr ? a.q_scale / (fmaxf(fabsf(a.nq[item] * a.q_scale), a.em[item]) + a.tiny) : 1.f;
+    for (int e = 0; e < 8; ++e) {
+        v[e] = live ? v[e] * f : 0.f;
+        ss = fmaf(v[e], v[e], ss);
     }
 #pragma unroll
-    for (int x = 0; x < ITEMS; ++x) {
-        v[x].x *= f[x]; v[x].y *= f[x]; v[x].z *= f[x]; v[x].w *= f[x];
-        const float ss = warp_sum(fmaf(v[x].x, v[x].x, fmaf(v[x].y, v[x].y, fmaf(v[x].z, v[x].z, v[x].w * v[x].w))));
-        const float r = 1.0f / sqrtf(ss / (float)a.V + a.eps) * a.post;
-        float y[4] = {v[x].x * r * w[x].x, v[x].y * r * w[x].y, v[x].z * r * w[x].z, v[x].w * r * w[x].w};
-        if (a.gate != nullptr) {
-            y[0] *= gs_sigmoid(g[x].x); y[1] *= gs_sigmoid(g[x].y); y[2] *= gs_sigmoid(g[x].z); y[3] *= gs_sigmoid(g[x].w);
-        }
-        if (in && item0 + x < items) gs_store4<T>(out + at[x], y[0], y[1], y[2], y[3]);
+    for (int off = LANES / 2; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+    const float r = 1.0f / sqrtf(ss / (float)a.V + a.eps) * a.post;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+        v[e] = v[e] * r * w[e];
+        if (a.gate != nullptr) v[e] *= gs_sigmoid(g[e]);
     }
+    if (live) gs_store8(out + (int64_t)row * a.out_ld + (int64_t)head * a.V + i, v);
 }
 
 // ----------------------------------------------------------------------------------------
@@ -771,19 +773,22 @@ X0NE_API int x0ne_scan_head_norm(HeadNormArgs a, void* out, int dt, int n_rows, 
     X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "scan_head_norm: unknown dtype tag %d", dt);
     if (n_rows == 0) return 0;
     const int64_t items = (int64_t)n_rows * a.heads;
-    const bool vec = a.V % 4 == 0 && a.V <= 128 && a.out_ld % 4 == 0 && a.gate_ld % 4 == 0 && gs_aligned16(a.o) && gs_aligned16(a.weight) &&
-                     gs_aligned16(a.gate) && (((uintptr_t)out) & (dt == X0NE_F32 ? 15 : 7)) == 0;
-    // (a head's sum runs over the same lanes in the same order however many heads a warp has)
-    const int per_warp = vec && items >= 4096 ? 4 : 1;
-    const dim3 grid((unsigned)((items + 4 * per_warp - 1) / (4 * per_warp))), block(128);
-#define GS_HEAD_NORM(T)                                                                                                  \
-    do {                                                                                                                 \
-        if (!vec) x0ne_launch(scan_head_norm_kernel<T>, grid, block, 0, stream, a, (T*)out, items);                      \
-        else if (per_warp == 4) x0ne_launch(scan_head_norm_vec_kernel<T, 4>, grid, block, 0, stream, a, (T*)out, items); \
-        else x0ne_launch(scan_head_norm_vec_kernel<T, 1>, grid, block, 0, stream, a, (T*)out, items);                    \
+    X0NE_REQUIRE(items < (1ll << 31), "scan_head_norm: %lld heads in all", (long long)items);
+    const bool vec = a.V % 8 == 0 && a.V <= 256 && a.out_ld % 8 == 0 && a.gate_ld % 4 == 0 && gs_aligned16(a.o) && gs_aligned16(a.weight) &&
+                     gs_aligned16(a.gate) && gs_aligned16(out);
+    const dim3 block(128);
+#define GS_HEAD_NORM_VEC(T, L) x0ne_launch(scan_head_norm_vec_kernel<T, L>, dim3((unsigned)((items * L + 127) / 128)), block, 0, stream, a, (T*)out, (uint32_t)items)
+#define GS_HEAD_NORM(T)                                                                                                                             \
+    do {                                                                                                                                            \
+        if (!vec) x0ne_launch(scan_head_norm_kernel<T>, dim3((unsigned)((items + 3) / 4)), block, 0, stream, a, (T*)out, (uint32_t)items);          \
+        else if (a.V <= 32) GS_HEAD_NORM_VEC(T, 4);                                                                                                 \
+        else if (a.V <= 64) GS_HEAD_NORM_VEC(T, 8);                                                                                                 \
+        else if (a.V <= 128) GS_HEAD_NORM_VEC(T, 16);                                                                                               \
+        else GS_HEAD_NORM_VEC(T, 32);                                                                                                               \
     } while (0)
     if (dt == X0NE_F32) GS_HEAD_NORM(float);
     else GS_HEAD_NORM(bf16);
 #undef GS_HEAD_NORM
+#undef GS_HEAD_NORM_VEC
     X0NE_LAUNCH_CHECK();
 }

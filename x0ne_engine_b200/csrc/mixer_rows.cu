@@ -962,9 +962,9 @@ __global__ void head_norm_rope_kv_write_kernel(HeadRopeArgs a, T* __restrict__ q
     pdl_prologue();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int heads = a.q_heads + 2 * cache.kv_heads;
-    const int64_t item = (int64_t)blockIdx.x * (blockDim.x >> 5) + warp;
-    if (item >= (int64_t)a.n_rows * heads) return;
-    const int row = (int)(item / heads), head = (int)(item - (int64_t)row * heads);
+    const uint32_t item = blockIdx.x * (blockDim.x >> 5) + warp;
+    if (item >= (uint32_t)a.n_rows * heads) return;
+    const int row = (int)(item / (uint32_t)heads), head = (int)(item - (uint32_t)row * heads);
     const int pos = a.row_pos[row];
     const float* src = a.src + (int64_t)row * a.ld;
     if (head >= a.q_heads + cache.kv_heads) {           // a value head
@@ -1072,6 +1072,7 @@ X0NE_API int x0ne_head_norm_rope_kv_write(HeadRopeArgs a, void* q_out, int dt, P
     X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "head_norm_rope: unknown dtype tag %d", dt);
     if (a.n_rows == 0) return 0;
     const int64_t items = (int64_t)a.n_rows * (a.q_heads + 2 * cache.kv_heads);
+    X0NE_REQUIRE(items < (1ll << 31), "head_norm_rope: %lld heads in all", (long long)items);
     const dim3 grid((unsigned)((items + 3) / 4)), block(128);
     const size_t smem = (size_t)4 * a.rot * sizeof(float);
     const bool vec = a.dim % 4 == 0 && (a.rot / 2) % 4 == 0 && cache_v_dim(cache) % 4 == 0 && a.ld % 4 == 0 && a.q_col % 4 == 0 && a.k_col % 4 == 0 &&
