@@ -22,7 +22,8 @@
 
 // exp(a * b) for a * b <= 0, closer than the library's exponential (whose error of up to two units in the last place, met
 // again at every token, is what a slowly decaying state adds up): the product's own rounding error is carried along
-// (x_lo), x = n ln2 + r with ln2 in two parts, and exp(r) is a polynomial of degree 7 over |r| <= ln2 / 2, all in fused
+// (x_lo), x = n ln2 + r with ln2 in two parts (the reduction of Cody and Waite, Software Manual for the Elementary
+// Functions), and exp(r) is the Taylor polynomial of degree 7 over |r| <= ln2 / 2, all in fused
 // multiply-adds.  Below 2^-126 the result is zero.
 __device__ __forceinline__ float ssm_exp_prod(float a, float b) {
     const float x = a * b;
