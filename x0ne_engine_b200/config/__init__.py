@@ -13,13 +13,16 @@ from .barorax import ARCHITECTURE as _BARORAX, MODEL_TYPE as _BARORAX_TYPE, Baro
 
 from .ravapel import ARCHITECTURE as _RAVAPEL, MODEL_TYPE as _RAVAPEL_TYPE, RavapelConfig
 
+from .tarudra import ARCHITECTURE as _TARUDRA, MODEL_TYPE as _TARUDRA_TYPE, TarudraConfig
+
 register_architecture(_QWEN3, _QWEN3_TYPE, Qwen3Config)
 register_architecture(_TENETAR, _TENETAR_TYPE, TenetarConfig)
 register_architecture(_ROVURAX, _ROVURAX_TYPE, RovuraxConfig)
 register_architecture(_RETUVIK, _RETUVIK_TYPE, RetuvikConfig)
 register_architecture(_BARORAX, _BARORAX_TYPE, BaroraxConfig)
 register_architecture(_RAVAPEL, _RAVAPEL_TYPE, RavapelConfig)
+register_architecture(_TARUDRA, _TARUDRA_TYPE, TarudraConfig)
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "Qwen3Config", "RovuraxConfig", "TenetarConfig", "RetuvikConfig", "BaroraxConfig",
-           "RavapelConfig",            "architectures", "config_from_dict", "config_from_folder", "detect",
+           "RavapelConfig", "TarudraConfig", "architectures", "config_from_dict", "config_from_folder", "detect",
            "register_architecture", "spec_from_folder", "unregister_architecture"]

@@ -188,6 +188,7 @@ __host__ __device__ __forceinline__ int cache_v_dim(const PagedCache& c) { retur
 struct GluParams {
     float limit, slope, shift;
     const float* bias;
+    int32_t out_act;            // products without a gate: what the epilogue does to a result (X0NE_OUT_*)
 };
 __device__ __forceinline__ float glu_act(float g, float u, const GluParams& p) {
     if (p.limit > 0.f) {
@@ -205,6 +206,19 @@ __device__ __forceinline__ float glu_act_at(float g, float u, int n, int N, cons
         u += __ldg(p.bias + N + at);
     }
     return glu_act(g, u, p);
+}
+
+// What a plain product's epilogue may do to a result before it is stored.
+#define X0NE_OUT_AS_IT_IS 0
+#define X0NE_OUT_RELU2 1        // max(v, 0)^2
+#define X0NE_OUT_SOFT_CAP 2     // limit * tanh(v / limit)
+__device__ __forceinline__ float soft_capped(float v, float cap) { return cap * tanhf(v / cap); }
+__device__ __forceinline__ float out_act(float v, const GluParams& p) {
+    if (p.out_act == X0NE_OUT_RELU2) {
+        v = fmaxf(v, 0.f);
+        return v * v;
+    }
+    return p.out_act == X0NE_OUT_SOFT_CAP ? soft_capped(v, p.limit) : v;
 }
 
 // What an attention kernel may be asked for beyond causal softmax over a window.  All zero: nothing.

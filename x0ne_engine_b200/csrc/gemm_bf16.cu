@@ -179,6 +179,7 @@ __global__ void __launch_bounds__(SM_WARPS * 32) gemm_smallm_kernel(const bf16* 
             if (n < N && m < M) {
                 float out = v[0];
                 if (SWIGLU) out = glu_act_at(v[0], v[SETS - 1], n, N, glu);
+                else out = out_act(out, glu);
                 Y[(int64_t)m * ldy + n] = from_f32<OutT>(out);
             }
         }
@@ -221,10 +222,7 @@ static int launch_smallm(const bf16* W, const bf16* X, OutT* Y, int M, int N, in
 
 // out_kind: 0 = bfloat16, 1 = float32, 2 = bfloat16 with SwiGLU over the packed [gate; up] weight
 // (W then has 2*N rows and y has N columns).
-// With out_kind 2, (limit, slope, shift, bias) choose the gated activation (`GluParams`; limit 0: SwiGLU; bias may be null).
-X0NE_API int x0ne_gemm_bf16_smallm_glu(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,
-                                       int sms, float limit, float slope, float shift, const float* bias, cudaStream_t stream) {
-    const GluParams glu = {limit, slope, shift, bias};
+static int smallm_dispatch(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind, int sms, GluParams glu, cudaStream_t stream) {
     X0NE_REQUIRE(M >= 0 && M <= 32 && N > 0 && K > 0, "gemm_smallm: M %d (at most 32) N %d K %d", M, N, K);
     X0NE_REQUIRE(K % 8 == 0, "gemm_smallm: K %d is not a multiple of 8", K);
     X0NE_REQUIRE(ldy >= N && sms > 0 && out_kind >= 0 && out_kind <= 2, "gemm_smallm: ldy %d N %d kind %d", ldy, N, out_kind);
@@ -241,6 +239,19 @@ X0NE_API int x0ne_gemm_bf16_smallm_glu(const void* W, const void* X, void* Y, in
     if (mt == 2) { X0NE_SMALLM(2) }
     { X0NE_SMALLM(4) }
 #undef X0NE_SMALLM
+}
+
+// With out_kind 2, (limit, slope, shift, bias) choose the gated activation (`GluParams`; limit 0: SwiGLU; bias may be null).
+X0NE_API int x0ne_gemm_bf16_smallm_glu(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,
+                                       int sms, float limit, float slope, float shift, const float* bias, cudaStream_t stream) {
+    return smallm_dispatch(W, X, Y, M, N, K, ldy, out_kind, sms, GluParams{limit, slope, shift, bias, 0}, stream);
+}
+
+// out_kind 0 or 1 with an activation of the result in the epilogue (X0NE_OUT_*; `limit`: the soft cap's).
+X0NE_API int x0ne_gemm_bf16_smallm_act(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind, int sms, int out_act,
+                                       float limit, cudaStream_t stream) {
+    X0NE_REQUIRE(out_kind <= 1 && out_act >= 0 && out_act <= 2 && (out_act != X0NE_OUT_SOFT_CAP || limit > 0.f), "gemm_smallm: activation %d of output kind %d", out_act, out_kind);
+    return smallm_dispatch(W, X, Y, M, N, K, ldy, out_kind, sms, GluParams{limit, 0.f, 0.f, nullptr, out_act}, stream);
 }
 
 X0NE_API int x0ne_gemm_bf16_smallm(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,

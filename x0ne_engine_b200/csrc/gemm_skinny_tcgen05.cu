@@ -216,6 +216,9 @@ __global__ void __launch_bounds__(SK_THREADS, 2) gemm_skinny_tc_kernel(const __g
                 const float u4[4] = {us.x, us.y, us.z, us.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i) o4[i] = glu_act_at(o4[i], u4[i], n0 + c + i, N, glu);
+            } else if (glu.out_act != X0NE_OUT_AS_IT_IS) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) o4[i] = out_act(o4[i], glu);
             }
             const int n = n0 + c;
             OutT* dst = Y + (int64_t)m * ldy + n;
@@ -289,10 +292,8 @@ static int launch_skinny(const void* W, const void* X, int x_rows, OutT* Y, int 
 // out_kind: 0 = bfloat16, 1 = float32, 2 = bfloat16 with SwiGLU over the packed [gate; up] weight
 // (W then has 2*N rows and y has N columns).  `status` as for the other tcgen05 kernels.
 // `x_rows`: rows allocated behind X (at least M).
-// With out_kind 2, (limit, slope, shift, bias) choose the gated activation (`GluParams`; limit 0: SwiGLU; bias may be null).
-X0NE_API int x0ne_gemm_bf16_skinny_tcgen05_glu(const void* W, const void* X, int x_rows, void* Y, int M, int N, int K, int ldy,
-                                               int out_kind, int* status, float limit, float slope, float shift, const float* bias, cudaStream_t stream) {
-    const GluParams glu = {limit, slope, shift, bias};
+static int skinny_dispatch(const void* W, const void* X, int x_rows, void* Y, int M, int N, int K, int ldy, int out_kind, int* status, GluParams glu,
+                           cudaStream_t stream) {
     X0NE_REQUIRE(M >= 0 && M <= 64 && N > 0 && K > 0 && x_rows >= M, "gemm_skinny_tc: M %d (at most 64, x has %d rows) N %d K %d", M, x_rows, N, K);
     X0NE_REQUIRE(K % 8 == 0, "gemm_skinny_tc: K %d is not a multiple of 8 (rows must be 16-byte aligned for TMA)", K);
     X0NE_REQUIRE(ldy >= N && out_kind >= 0 && out_kind <= 2 && status != nullptr, "gemm_skinny_tc: ldy %d N %d kind %d", ldy, N, out_kind);
@@ -301,6 +302,19 @@ X0NE_API int x0ne_gemm_bf16_skinny_tcgen05_glu(const void* W, const void* X, int
     if (out_kind == 0) return launch_skinny<false, bf16>(W, X, x_rows, (bf16*)Y, M, N, K, ldy, status, glu, stream);
     if (out_kind == 1) return launch_skinny<false, float>(W, X, x_rows, (float*)Y, M, N, K, ldy, status, glu, stream);
     return launch_skinny<true, bf16>(W, X, x_rows, (bf16*)Y, M, N, K, ldy, status, glu, stream);
+}
+
+// With out_kind 2, (limit, slope, shift, bias) choose the gated activation (`GluParams`; limit 0: SwiGLU; bias may be null).
+X0NE_API int x0ne_gemm_bf16_skinny_tcgen05_glu(const void* W, const void* X, int x_rows, void* Y, int M, int N, int K, int ldy,
+                                               int out_kind, int* status, float limit, float slope, float shift, const float* bias, cudaStream_t stream) {
+    return skinny_dispatch(W, X, x_rows, Y, M, N, K, ldy, out_kind, status, GluParams{limit, slope, shift, bias, 0}, stream);
+}
+
+// out_kind 0 or 1 with an activation of the result in the epilogue (X0NE_OUT_*; `limit`: the soft cap's).
+X0NE_API int x0ne_gemm_bf16_skinny_tcgen05_act(const void* W, const void* X, int x_rows, void* Y, int M, int N, int K, int ldy, int out_kind, int* status,
+                                               int out_act, float limit, cudaStream_t stream) {
+    X0NE_REQUIRE(out_kind <= 1 && out_act >= 0 && out_act <= 2 && (out_act != X0NE_OUT_SOFT_CAP || limit > 0.f), "gemm_skinny_tc: activation %d of output kind %d", out_act, out_kind);
+    return skinny_dispatch(W, X, x_rows, Y, M, N, K, ldy, out_kind, status, GluParams{limit, 0.f, 0.f, nullptr, out_act}, stream);
 }
 
 X0NE_API int x0ne_gemm_bf16_skinny_tcgen05(const void* W, const void* X, int x_rows, void* Y, int M, int N, int K, int ldy,

@@ -192,6 +192,9 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_kernel(const __grid_consta
                     if (glu.bias != nullptr) tc_add_bias(v, u, &sh->bias[quarter][c * 32]);
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = glu_act(v[i], u[i], glu);
+                } else if (glu.out_act != X0NE_OUT_AS_IT_IS) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] = out_act(v[i], glu);
                 }
                 const int n = n0 + c * 32;
                 if (m < M) {
@@ -395,6 +398,9 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_pair_kernel(const __grid_c
                     if (glu.bias != nullptr) tc_add_bias(v, u, &sh->bias[quarter][c * 32]);
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = glu_act(v[i], u[i], glu);
+                } else if (glu.out_act != X0NE_OUT_AS_IT_IS) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] = out_act(v[i], glu);
                 }
                 const int n = n0 + c * 32;
                 if (m < M) {
@@ -529,10 +535,7 @@ static int launch_tc_pair(const void* W, const void* X, OutT* Y, int M, int N, i
 // first call; a non-zero value afterwards says a barrier wait ran out (1 copy, 2 MMA, 3 epilogue)
 // and the output is not valid.
 // `pair` = 1 uses pairs of blocks (256 x 256 tiles), 0 single blocks (128 x 256 tiles).
-// With out_kind 2, (limit, slope, shift, bias) choose the gated activation (`GluParams`; limit 0: SwiGLU; bias may be null).
-X0NE_API int x0ne_gemm_bf16_tcgen05_glu(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,
-                                        int pair, int* status, float limit, float slope, float shift, const float* bias, cudaStream_t stream) {
-    const GluParams glu = {limit, slope, shift, bias};
+static int tc_dispatch(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind, int pair, int* status, GluParams glu, cudaStream_t stream) {
     X0NE_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tc: M %d N %d K %d", M, N, K);
     X0NE_REQUIRE(K % 8 == 0, "gemm_tc: K %d is not a multiple of 8 (rows must be 16-byte aligned)", K);
     X0NE_REQUIRE(ldy >= N && out_kind >= 0 && out_kind <= 2 && status != nullptr, "gemm_tc: ldy %d N %d kind %d", ldy, N, out_kind);
@@ -545,6 +548,19 @@ X0NE_API int x0ne_gemm_bf16_tcgen05_glu(const void* W, const void* X, void* Y, i
     if (out_kind == 0) return launch_tc<false, bf16>(W, X, (bf16*)Y, M, N, K, ldy, status, glu, stream);
     if (out_kind == 1) return launch_tc<false, float>(W, X, (float*)Y, M, N, K, ldy, status, glu, stream);
     return launch_tc<true, bf16>(W, X, (bf16*)Y, M, N, K, ldy, status, glu, stream);
+}
+
+// With out_kind 2, (limit, slope, shift, bias) choose the gated activation (`GluParams`; limit 0: SwiGLU; bias may be null).
+X0NE_API int x0ne_gemm_bf16_tcgen05_glu(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,
+                                        int pair, int* status, float limit, float slope, float shift, const float* bias, cudaStream_t stream) {
+    return tc_dispatch(W, X, Y, M, N, K, ldy, out_kind, pair, status, GluParams{limit, slope, shift, bias, 0}, stream);
+}
+
+// out_kind 0 or 1 with an activation of the result in the epilogue (X0NE_OUT_*; `limit`: the soft cap's).
+X0NE_API int x0ne_gemm_bf16_tcgen05_act(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind, int pair, int* status,
+                                        int out_act, float limit, cudaStream_t stream) {
+    X0NE_REQUIRE(out_kind <= 1 && out_act >= 0 && out_act <= 2 && (out_act != X0NE_OUT_SOFT_CAP || limit > 0.f), "gemm_tc: activation %d of output kind %d", out_act, out_kind);
+    return tc_dispatch(W, X, Y, M, N, K, ldy, out_kind, pair, status, GluParams{limit, 0.f, 0.f, nullptr, out_act}, stream);
 }
 
 X0NE_API int x0ne_gemm_bf16_tcgen05(const void* W, const void* X, void* Y, int M, int N, int K, int ldy, int out_kind,

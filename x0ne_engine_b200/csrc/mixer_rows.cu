@@ -775,9 +775,10 @@ X0NE_API int x0ne_bias_act(const void* x, const float* bias, void* out, int dt, 
 // ----------------------------------------------------------------------------------------
 // Preparation of an attention that rotates interleaved pairs and may hold several score maps per head.  src holds, per
 // row, the queries at column 0 (q_heads x maps x dim), the keys at k_col (kv_heads x maps x dim) and the values at v_col
-// (kv_heads x value width).  Of every (head, map) the first `rot` values are pairs (2i, 2i + 1) that turn by
-// pos * freq[i]: (u, v) -> (u cos - v sin, v cos + u sin); `table` (float32 [positions][rot]: rot/2 cosines, then rot/2
-// sines) replaces the computation for the positions it covers.  With unit_eps >= 0 every (head, map), after its rotation,
+// (kv_heads x value width); `bias` (float32, one value per column of src, or null) is added first, to the values too.  Of
+// every (head, map) the first `rot` values are pairs (2i, 2i + 1) that turn by pos * freq[i]: (u, v) -> (u cos - v sin, v cos
+// + u sin); `table` (float32 [positions][rot]: rot/2 cosines, then rot/2
+// sines) replaces the computation for the positions it covers; computed cosines and sines are multiplied by `mag`.  With unit_eps >= 0 every (head, map), after its rotation,
 // is divided by sqrt(mean(x^2) + unit_eps) over its dim values.  A kv head's maps lie side by side in its key row of
 // maps x dim values.  Queries go to q_out as [rows][q_heads x maps][dim], or, with `q_padded`, as [rows][q_heads x maps]
 // [maps x dim] with map m's values at column m x dim and zeros beside them: such a query, met with the whole key row,
@@ -785,15 +786,15 @@ X0NE_API int x0ne_bias_act(const void* x, const float* bias, void* out, int dt, 
 // write no keys or values.
 // ----------------------------------------------------------------------------------------
 template <typename T>
-__global__ void rope_pairs_kv_write_kernel(const T* __restrict__ src, int ld, int k_col, int v_col, const float* __restrict__ freq,
-                                           const float* __restrict__ table, int table_positions, int rot, int maps, int dim,
+__global__ void rope_pairs_kv_write_kernel(const T* __restrict__ src, const float* __restrict__ bias, int ld, int k_col, int v_col, const float* __restrict__ freq,
+                                           const float* __restrict__ table, int table_positions, int rot, int maps, int dim, float mag,
                                            float unit_eps, T* __restrict__ q_out, int q_heads, int q_padded, PagedCache cache,
                                            const int32_t* __restrict__ row_slot, const int32_t* __restrict__ row_pos, int n_rows,
                                            int write_kv) {
     pdl_prologue();
     const int lane = threadIdx.x & 31;
-    const int nq = q_heads * maps, nk = cache.kv_heads * maps;
-    const int units = nq + nk + cache.kv_heads;
+    const int nq = q_heads * maps, nk = write_kv ? cache.kv_heads * maps : 0;
+    const int units = nq + nk + (write_kv ? cache.kv_heads : 0);
     const int64_t item = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (item >= (int64_t)n_rows * units) return;
     const int row = (int)(item / units), unit = (int)(item % units);
@@ -804,12 +805,16 @@ __global__ void rope_pairs_kv_write_kernel(const T* __restrict__ src, int ld, in
         const int64_t off = write_kv ? cache_row_offset(cache, slot, pos, g, 1) : -1;
         if (off < 0) return;
         T* dst = (T*)cache.base + off;
-        for (int i = lane; i < vd; i += 32) dst[i] = s[v_col + (int64_t)g * vd + i];
+        for (int i = lane; i < vd; i += 32) {
+            const int col = v_col + g * vd + i;
+            dst[i] = bias != nullptr ? from_f32<T>(to_f32(s[col]) + bias[col]) : s[col];
+        }
         return;
     }
     const bool is_q = unit < nq;
     const int sub = is_q ? unit : unit - nq;      // head x maps + map
     const T* x = s + (is_q ? 0 : k_col) + (int64_t)sub * dim;
+    const float* b = bias != nullptr ? bias + (is_q ? 0 : k_col) + (int64_t)sub * dim : nullptr;
     T* dst;
     if (is_q) {
         const int w = q_padded ? maps * dim : dim;
@@ -832,6 +837,10 @@ __global__ void rope_pairs_kv_write_kernel(const T* __restrict__ src, int ld, in
         float ss = 0.f;
         for (int p = lane; p < pairs; p += 32) {
             float u = to_f32(x[2 * p]), v = 2 * p + 1 < dim ? to_f32(x[2 * p + 1]) : 0.f;
+            if (b != nullptr) {
+                u += b[2 * p];
+                if (2 * p + 1 < dim) v += b[2 * p + 1];
+            }
             if (p < half) {
                 float c, sn;
                 if (tabled) {
@@ -839,6 +848,8 @@ __global__ void rope_pairs_kv_write_kernel(const T* __restrict__ src, int ld, in
                     sn = table[(int64_t)pos * rot + half + p];
                 } else {
                     sincosf((float)pos * freq[p], &sn, &c);
+                    c *= mag;
+                    sn *= mag;
                 }
                 const float ru = u * c - v * sn, rv = v * c + u * sn;
                 u = ru;
@@ -856,8 +867,71 @@ __global__ void rope_pairs_kv_write_kernel(const T* __restrict__ src, int ld, in
     }
 }
 
-X0NE_API int x0ne_rope_pairs_kv_write(const void* src, int dt, int ld, int k_col, int v_col, const float* freq, const float* table,
-                                      int table_positions, int rot, int maps, int dim, float unit_eps, void* q_out, int q_heads,
+// The same for one map per head without unit norm, 8 values per thread: dim, rot, the value width, the row pitch and the
+// columns are multiples of 8.  A block takes 8 x blockDim.x values of a row.
+template <typename T>
+__global__ void __launch_bounds__(128) rope_pairs_kv_write_vec_kernel(const T* __restrict__ src, const float* __restrict__ bias, int ld, int k_col, int v_col,
+                                                                      const float* __restrict__ freq, const float* __restrict__ table, int table_positions,
+                                                                      int rot, int dim, float mag, T* __restrict__ q_out, int q_heads, PagedCache cache,
+                                                                      const int32_t* __restrict__ row_slot, const int32_t* __restrict__ row_pos, int write_kv) {
+    pdl_launch_dependents();
+    const int row = blockIdx.x, vd = cache_v_dim(cache);
+    const int nq = q_heads * dim, nk = write_kv ? cache.kv_heads * dim : 0, nv = write_kv ? cache.kv_heads * vd : 0;
+    const int i = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+    if (i >= nq + nk + nv) return;
+    const int pos = row_pos[row], slot = row_slot[row];
+    T* dst;
+    int col, d, width;
+    if (i < nq) {
+        col = i;
+        d = i % dim;
+        dst = q_out + (int64_t)row * nq + i;
+    } else {
+        const bool is_k = i < nq + nk;
+        const int e = i - (is_k ? nq : nq + nk);
+        width = is_k ? dim : vd;
+        col = (is_k ? k_col : v_col) + e;
+        const int64_t off = cache_row_offset(cache, slot, pos, e / width, is_k ? 0 : 1);
+        if (off < 0) return;
+        const int within = e % width;
+        d = is_k ? within : dim;               // (values do not turn)
+        dst = (T*)cache.base + off + within;
+    }
+    float c[4], sn[4], b[8];
+    if (d < rot) {
+        const int half = rot / 2, p = d / 2;
+        if (table != nullptr && pos >= 0 && pos < table_positions) {
+            const float4 c4 = *reinterpret_cast<const float4*>(table + (int64_t)pos * rot + p), s4 = *reinterpret_cast<const float4*>(table + (int64_t)pos * rot + half + p);
+            c[0] = c4.x; c[1] = c4.y; c[2] = c4.z; c[3] = c4.w;
+            sn[0] = s4.x; sn[1] = s4.y; sn[2] = s4.z; sn[3] = s4.w;
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                sincosf((float)pos * freq[p + e], &sn[e], &c[e]);
+                c[e] *= mag;
+                sn[e] *= mag;
+            }
+        }
+    }
+    if (bias != nullptr) load8f(bias + col, b);
+    pdl_wait();
+    float x[8];
+    load8f(src + (int64_t)row * ld + col, x);
+    if (bias != nullptr)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] += b[e];
+    if (d < rot)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float u = x[2 * e], v = x[2 * e + 1];
+            x[2 * e] = u * c[e] - v * sn[e];
+            x[2 * e + 1] = v * c[e] + u * sn[e];
+        }
+    store8f(dst, x);
+}
+
+X0NE_API int x0ne_rope_pairs_kv_write(const void* src, const float* bias, int dt, int ld, int k_col, int v_col, const float* freq, const float* table,
+                                      int table_positions, int rot, int maps, int dim, float mag, float unit_eps, void* q_out, int q_heads,
                                       int q_padded, PagedCache cache, const int32_t* row_slot, const int32_t* row_pos, int n_rows,
                                       int write_kv, cudaStream_t stream) {
     X0NE_REQUIRE(n_rows >= 0 && q_heads > 0 && maps > 0 && dim > 0 && rot >= 0 && rot % 2 == 0 && rot <= dim && cache.kv_heads > 0,
@@ -865,21 +939,34 @@ X0NE_API int x0ne_rope_pairs_kv_write(const void* src, int dt, int ld, int k_col
     X0NE_REQUIRE(cache.head_dim == maps * dim && cache.v_dim >= 0, "rope_pairs: the cache's key rows hold %d values, not %d maps of %d", cache.head_dim, maps, dim);
     X0NE_REQUIRE(rot == 0 || freq != nullptr, "rope_pairs: no frequencies");
     const int vd = cache_v_dim(cache);
-    X0NE_REQUIRE(k_col >= q_heads * maps * dim && v_col >= k_col + cache.kv_heads * maps * dim && ld >= v_col + cache.kv_heads * vd,
+    X0NE_REQUIRE(ld >= q_heads * maps * dim && (!write_kv || (k_col >= q_heads * maps * dim && v_col >= k_col + cache.kv_heads * maps * dim && ld >= v_col + cache.kv_heads * vd)),
                  "rope_pairs: columns %d, %d do not fit rows of %d", k_col, v_col, ld);
+    X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "rope_pairs: unknown dtype tag %d", dt);
     if (n_rows == 0) return 0;
+    const bool vec = maps == 1 && unit_eps < 0.f && !q_padded && dim % 8 == 0 && rot % 8 == 0 && ld % 8 == 0 &&
+                     (!write_kv || (vd % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 && cache.page_stride % 8 == 0 && ((uintptr_t)cache.base & 15) == 0)) &&
+                     ((((uintptr_t)src | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)table) & 15) == 0);
+    if (vec) {
+        const int pieces = (q_heads * dim + (write_kv ? cache.kv_heads * (dim + vd) : 0)) / 8;
+        const dim3 vgrid(n_rows, (pieces + 127) / 128), vblock(128);
+        if (dt == X0NE_F32)
+            x0ne_launch(rope_pairs_kv_write_vec_kernel<float>, vgrid, vblock, 0, stream, (const float*)src, bias, ld, k_col, v_col, freq, table, table_positions, rot,
+                        dim, mag, (float*)q_out, q_heads, cache, row_slot, row_pos, write_kv);
+        else
+            x0ne_launch(rope_pairs_kv_write_vec_kernel<bf16>, vgrid, vblock, 0, stream, (const bf16*)src, bias, ld, k_col, v_col, freq, table, table_positions, rot,
+                        dim, mag, (bf16*)q_out, q_heads, cache, row_slot, row_pos, write_kv);
+        X0NE_LAUNCH_CHECK();
+    }
     const int warps = 4;
-    const int64_t items = (int64_t)n_rows * (q_heads * maps + cache.kv_heads * maps + cache.kv_heads);
+    const int64_t items = (int64_t)n_rows * (q_heads * maps + (write_kv ? cache.kv_heads * maps + cache.kv_heads : 0));
     X0NE_REQUIRE((items + warps - 1) / warps <= 0x7fffffff, "rope_pairs: too many rows");
     const dim3 grid((unsigned)((items + warps - 1) / warps));
     if (dt == X0NE_F32)
-        x0ne_launch(rope_pairs_kv_write_kernel<float>, grid, dim3(warps * 32), 0, stream, (const float*)src, ld, k_col, v_col, freq, table,
-                    table_positions, rot, maps, dim, unit_eps, (float*)q_out, q_heads, q_padded, cache, row_slot, row_pos, n_rows, write_kv);
-    else if (dt == X0NE_BF16)
-        x0ne_launch(rope_pairs_kv_write_kernel<bf16>, grid, dim3(warps * 32), 0, stream, (const bf16*)src, ld, k_col, v_col, freq, table,
-                    table_positions, rot, maps, dim, unit_eps, (bf16*)q_out, q_heads, q_padded, cache, row_slot, row_pos, n_rows, write_kv);
+        x0ne_launch(rope_pairs_kv_write_kernel<float>, grid, dim3(warps * 32), 0, stream, (const float*)src, bias, ld, k_col, v_col, freq, table,
+                    table_positions, rot, maps, dim, mag, unit_eps, (float*)q_out, q_heads, q_padded, cache, row_slot, row_pos, n_rows, write_kv);
     else
-        X0NE_REQUIRE(false, "rope_pairs: unknown dtype tag %d", dt);
+        x0ne_launch(rope_pairs_kv_write_kernel<bf16>, grid, dim3(warps * 32), 0, stream, (const bf16*)src, bias, ld, k_col, v_col, freq, table,
+                    table_positions, rot, maps, dim, mag, unit_eps, (bf16*)q_out, q_heads, q_padded, cache, row_slot, row_pos, n_rows, write_kv);
     X0NE_LAUNCH_CHECK();
 }
 
@@ -1085,5 +1172,231 @@ X0NE_API int x0ne_head_norm_rope_kv_write(HeadRopeArgs a, void* q_out, int dt, P
         if (vec) x0ne_launch(head_norm_rope_kv_write_kernel<bf16, true>, grid, block, smem, stream, a, (bf16*)q_out, cache);
         else x0ne_launch(head_norm_rope_kv_write_kernel<bf16, false>, grid, block, smem, stream, a, (bf16*)q_out, cache);
     }
+    X0NE_LAUNCH_CHECK();
+}
+
+// ----------------------------------------------------------------------------------------
+// Latent attention whose queries go through a latent of their own, or whose rotated parts turn in halves.  Two kernels around
+// the products that need what the first one makes:
+//   latent_rows:     c_q = RMS norm of `q_rank` values at dq_col (weight norm_q)        -> cq_out [rows][q_rank]   (q_rank 0: none)
+//                    c   = RMS norm of `rank` values at dkv_col (weight norm_kv)        -> cache row [0, rank)
+//                    the `rot` values behind them, turned                              -> cache row [rank, rank + rot)
+//   latent_queries:  q_out[row][head] = [ q_abs[head][row][0 .. rank) | turned q[row][head][dim .. dim + rot) ]
+// Pairs: (i, i + rot/2) where `half_layout`, else (2i, 2i + 1); pair i turns by pos * freq[i], cosines and sines times `mag`;
+// `table` (float32 [positions][rot]: rot/2 cosines, then rot/2 sines, scaled) replaces the computation for the positions it
+// covers.  latent_rows: a warp per (row, one of the two norms); latent_queries: a thread per piece of 8 (or 1) latent values or
+// per rotated pair.  Norms, angles and the rotation are float32, one rounding at the store.
+// ----------------------------------------------------------------------------------------
+struct LatentTurn {
+    const float* freq;
+    const float* table;
+    float mag;
+    int32_t table_positions, rot, half_layout;
+};
+__device__ __forceinline__ void latent_turn(const LatentTurn& t, int pos, int i, float& c, float& s) {
+    if (t.table != nullptr && pos >= 0 && pos < t.table_positions) {
+        c = t.table[(int64_t)pos * t.rot + i];
+        s = t.table[(int64_t)pos * t.rot + t.rot / 2 + i];
+    } else {
+        sincosf((float)pos * t.freq[i], &s, &c);
+        c *= t.mag;
+        s *= t.mag;
+    }
+}
+
+struct LatentRowsArgs {
+    const void* src;
+    int64_t ld;
+    int32_t dq_col, q_rank, dkv_col, rank;
+    const float* norm_q;
+    const float* norm_kv;
+    float eps;
+    LatentTurn turn;
+    const int32_t* row_slot;
+    const int32_t* row_pos;
+    int32_t n_rows, write_cache;
+};
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(128) latent_rows_kernel(LatentRowsArgs a, T* __restrict__ cq_out, PagedCache cache) {
+    pdl_prologue();
+    const int lane = threadIdx.x & 31;
+    const int item = blockIdx.x * 4 + (threadIdx.x >> 5), row = item >> 1;
+    if (row >= a.n_rows) return;
+    const bool is_q = (item & 1) == 0;
+    const T* s = (const T*)a.src + (int64_t)row * a.ld + (is_q ? a.dq_col : a.dkv_col);
+    const int n = is_q ? a.q_rank : a.rank;
+    const float* w = is_q ? a.norm_q : a.norm_kv;
+    T* dst;
+    const int pos = a.row_pos[row];
+    if (is_q) {
+        if (n == 0) return;
+        dst = cq_out + (int64_t)row * n;
+    } else {
+        const int64_t off = a.write_cache ? cache_row_offset(cache, a.row_slot[row], pos, 0, 0) : -1;
+        if (off < 0) return;
+        dst = (T*)cache.base + off;
+    }
+    float ss = 0.f;
+    if (VEC) {
+        for (int i = 8 * lane; i < n; i += 256) {
+            float x[8];
+            load8f(s + i, x);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
+        }
+    } else {
+        for (int i = lane; i < n; i += 32) {
+            const float x = to_f32(s[i]);
+            ss = fmaf(x, x, ss);
+        }
+    }
+    const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
+    if (VEC) {
+        for (int i = 8 * lane; i < n; i += 256) {
+            float x[8], wv[8];
+            load8f(s + i, x);
+            load8f(w + i, wv);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = x[e] * scale * wv[e];
+            store8f(dst + i, x);
+        }
+    } else {
+        for (int i = lane; i < n; i += 32) dst[i] = from_f32<T>(to_f32(s[i]) * scale * w[i]);
+    }
+    if (is_q) return;
+    const int half = a.turn.rot / 2;
+    for (int i = lane; i < half; i += 32) {
+        const int iu = n + (a.turn.half_layout ? i : 2 * i), iv = n + (a.turn.half_layout ? i + half : 2 * i + 1);
+        const float u = to_f32(s[iu]), v = to_f32(s[iv]);
+        float c, sn;
+        latent_turn(a.turn, pos, i, c, sn);
+        dst[iu] = from_f32<T>(u * c - v * sn);
+        dst[iv] = from_f32<T>(v * c + u * sn);
+    }
+}
+
+X0NE_API int x0ne_latent_rows(LatentRowsArgs a, void* cq_out, int dt, PagedCache cache, cudaStream_t stream) {
+    X0NE_REQUIRE(a.n_rows >= 0 && a.n_rows < (1 << 29) && a.q_rank >= 0 && a.rank > 0 && a.turn.rot >= 0 && a.turn.rot % 2 == 0 && (a.turn.rot == 0 || a.turn.freq != nullptr),
+                 "latent_rows: ranks %d, %d, %d rotated values", a.q_rank, a.rank, a.turn.rot);
+    X0NE_REQUIRE(cache.kv_heads == 1 && cache.head_dim == a.rank + a.turn.rot, "latent_rows: the cache row is %d x %d, not 1 x %d", cache.kv_heads, cache.head_dim, a.rank + a.turn.rot);
+    X0NE_REQUIRE(a.dq_col >= 0 && a.dkv_col >= 0 && a.dq_col + a.q_rank <= a.ld && a.dkv_col + a.rank + a.turn.rot <= a.ld && a.norm_kv != nullptr &&
+                     (a.q_rank == 0 || (a.norm_q != nullptr && cq_out != nullptr)), "latent_rows: columns lie outside the source rows, or a tensor is missing");
+    X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "latent_rows: unknown dtype tag %d", dt);
+    if (a.n_rows == 0) return 0;
+    const bool vec = a.q_rank % 8 == 0 && a.rank % 8 == 0 && a.ld % 8 == 0 && a.dq_col % 8 == 0 && a.dkv_col % 8 == 0 && cache.head_dim % 8 == 0 && cache.page_stride % 8 == 0 &&
+                     ((((uintptr_t)a.src | (uintptr_t)a.norm_q | (uintptr_t)a.norm_kv | (uintptr_t)cq_out | (uintptr_t)cache.base) & 15) == 0);
+    const dim3 grid((unsigned)((a.n_rows + 1) / 2)), block(128);
+#define LATENT_ROWS(T, VEC) x0ne_launch(latent_rows_kernel<T, VEC>, grid, block, 0, stream, a, (T*)cq_out, cache)
+    if (dt == X0NE_F32) {
+        if (vec) LATENT_ROWS(float, true); else LATENT_ROWS(float, false);
+    } else {
+        if (vec) LATENT_ROWS(bf16, true); else LATENT_ROWS(bf16, false);
+    }
+#undef LATENT_ROWS
+    X0NE_LAUNCH_CHECK();
+}
+
+// q: [rows][q_ld], head h at column h * (dim + rot); q_abs: [heads][head_stride] of rows of `rank` values.
+template <typename T, int PIECE>
+__global__ void __launch_bounds__(128) latent_queries_kernel(const T* __restrict__ q, int64_t q_ld, const T* __restrict__ q_abs, int64_t head_stride, LatentTurn turn,
+                                                             const int32_t* __restrict__ row_pos, T* __restrict__ q_out, int heads, int dim, int rank) {
+    pdl_launch_dependents();
+    const int row = blockIdx.x, pos = row_pos[row], half = turn.rot / 2, per_head = rank / PIECE, qw = rank + turn.rot;
+    const int i = blockIdx.y * blockDim.x + threadIdx.x, n_copy = heads * per_head;
+    if (i >= n_copy + heads * half) return;
+    float c = 0.f, sn = 0.f;
+    if (i >= n_copy) latent_turn(turn, pos, (i - n_copy) % half, c, sn);
+    pdl_wait();
+    T* qo = q_out + (int64_t)row * heads * qw;
+    if (i < n_copy) {
+        const int h = i / per_head, d = (i - h * per_head) * PIECE;
+        const T* from = q_abs + (int64_t)h * head_stride + (int64_t)row * rank + d;
+        if (PIECE == 8) copy8(qo + (int64_t)h * qw + d, from);
+        else qo[(int64_t)h * qw + d] = *from;
+        return;
+    }
+    const int e = i - n_copy, h = e / half, j = e - h * half;
+    const int iu = turn.half_layout ? j : 2 * j, iv = turn.half_layout ? j + half : 2 * j + 1;
+    const T* from = q + (int64_t)row * q_ld + (int64_t)h * (dim + turn.rot) + dim;
+    const float u = to_f32(from[iu]), v = to_f32(from[iv]);
+    T* to = qo + (int64_t)h * qw + rank;
+    to[iu] = from_f32<T>(u * c - v * sn);
+    to[iv] = from_f32<T>(v * c + u * sn);
+}
+
+X0NE_API int x0ne_latent_queries(const void* q, int64_t q_ld, const void* q_abs, int64_t head_stride, LatentTurn turn, const int32_t* row_pos, void* q_out, int dt,
+                                 int heads, int dim, int rank, int n_rows, cudaStream_t stream) {
+    X0NE_REQUIRE(n_rows >= 0 && heads > 0 && dim > 0 && rank > 0 && turn.rot >= 0 && turn.rot % 2 == 0 && (turn.rot == 0 || turn.freq != nullptr) &&
+                     q_ld >= (int64_t)heads * (dim + turn.rot) && head_stride >= (int64_t)n_rows * rank, "latent_queries: heads %d dim %d rot %d rank %d", heads, dim, turn.rot, rank);
+    X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "latent_queries: unknown dtype tag %d", dt);
+    if (n_rows == 0) return 0;
+    const bool vec = rank % 8 == 0 && turn.rot % 8 == 0 && head_stride % 8 == 0 && ((((uintptr_t)q_abs | (uintptr_t)q_out) & 15) == 0);
+    const int per_row = heads * (rank / (vec ? 8 : 1)) + heads * (turn.rot / 2);
+    const dim3 grid(n_rows, (per_row + 127) / 128), block(128);
+#define LATENT_QUERIES(T, P) x0ne_launch(latent_queries_kernel<T, P>, grid, block, 0, stream, (const T*)q, q_ld, (const T*)q_abs, head_stride, turn, row_pos, (T*)q_out, heads, dim, rank)
+    if (dt == X0NE_F32) {
+        if (vec) LATENT_QUERIES(float, 8); else LATENT_QUERIES(float, 1);
+    } else {
+        if (vec) LATENT_QUERIES(bf16, 8); else LATENT_QUERIES(bf16, 1);
+    }
+#undef LATENT_QUERIES
+    X0NE_LAUNCH_CHECK();
+}
+
+// ----------------------------------------------------------------------------------------
+// Heads side by side, gated: out[row][h * V + d] = x[h][row][d] * sigmoid(gate[row * gate_ld + h * V + d]), the heads' rows
+// head_stride values apart (what a product per head leaves).
+// ----------------------------------------------------------------------------------------
+template <typename T, int PIECE>
+__global__ void __launch_bounds__(128) heads_gate_kernel(const T* __restrict__ x, int64_t head_stride, const T* __restrict__ gate, int64_t gate_ld, T* __restrict__ out,
+                                                         int heads, int V) {
+    pdl_prologue();
+    const int row = blockIdx.x, i = (blockIdx.y * blockDim.x + threadIdx.x) * PIECE;
+    if (i >= heads * V) return;
+    const int h = i / V, d = i - h * V;
+    const T* from = x + (int64_t)h * head_stride + (int64_t)row * V + d;
+    const T* g = gate + (int64_t)row * gate_ld + i;
+    T* to = out + (int64_t)row * heads * V + i;
+    if (PIECE == 8) {
+        float a[8], b[8];
+        load8f(from, a);
+        load8f(g, b);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] /= 1.0f + expf(-b[e]);
+        store8f(to, a);
+    } else {
+        *to = from_f32<T>(to_f32(*from) / (1.0f + expf(-to_f32(*g))));
+    }
+}
+
+X0NE_API int x0ne_heads_gate(const void* x, int64_t head_stride, const void* gate, int64_t gate_ld, void* out, int dt, int n_rows, int heads, int V, cudaStream_t stream) {
+    X0NE_REQUIRE(n_rows >= 0 && heads > 0 && V > 0 && head_stride >= (int64_t)n_rows * V && gate_ld >= (int64_t)heads * V, "heads_gate: rows %d heads %d of %d", n_rows, heads, V);
+    X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "heads_gate: unknown dtype tag %d", dt);
+    if (n_rows == 0) return 0;
+    const bool vec = V % 8 == 0 && head_stride % 8 == 0 && gate_ld % 8 == 0 && ((((uintptr_t)x | (uintptr_t)gate | (uintptr_t)out) & 15) == 0);
+    const dim3 grid(n_rows, (heads * V / (vec ? 8 : 1) + 127) / 128), block(128);
+#define HEADS_GATE(T, P) x0ne_launch(heads_gate_kernel<T, P>, grid, block, 0, stream, (const T*)x, head_stride, (const T*)gate, gate_ld, (T*)out, heads, V)
+    if (dt == X0NE_F32) {
+        if (vec) HEADS_GATE(float, 8); else HEADS_GATE(float, 1);
+    } else {
+        if (vec) HEADS_GATE(bf16, 8); else HEADS_GATE(bf16, 1);
+    }
+#undef HEADS_GATE
+    X0NE_LAUNCH_CHECK();
+}
+
+// ----------------------------------------------------------------------------------------
+// x = cap tanh(x / cap) in place, float32.
+// ----------------------------------------------------------------------------------------
+__global__ void soft_cap_kernel(float* __restrict__ x, int64_t total, float cap) {
+    pdl_prologue();
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) x[i] = soft_capped(x[i], cap);
+}
+X0NE_API int x0ne_soft_cap(float* x, int64_t total, float cap, cudaStream_t stream) {
+    X0NE_REQUIRE(total >= 0 && cap > 0.f, "soft_cap: %lld values, cap %g", (long long)total, cap);
+    if (total == 0) return 0;
+    const int64_t blocks = (total + 255) / 256;
+    x0ne_launch(soft_cap_kernel, dim3((unsigned)(blocks < 148 * 32 ? blocks : 148 * 32)), dim3(256), 0, stream, x, total, cap);
     X0NE_LAUNCH_CHECK();
 }

@@ -133,6 +133,34 @@ class NormConvArg(Structure):
                 ("width", c_int32), ("taps", c_int32)]
 
 
+class DeltaArg(Structure):
+    """Mirror of `struct DeltaArgs` in delta_rule.cu."""
+    _fields_ = [("src", c_void_p), ("ld", c_int64), ("q_col", c_int32), ("k_col", c_int32), ("v_col", c_int32), ("a_col", c_int32),
+                ("b_col", c_int32), ("g_col", c_int32), ("conv", c_void_p), ("A", c_void_p), ("dt_bias", c_void_p), ("norm_w", c_void_p),
+                ("q_scale", c_float), ("eps", c_float), ("state", c_void_p), ("state_stride", c_int64), ("ring_off", c_int64),
+                ("row_slot", c_void_p), ("row_pos", c_void_p), ("seq_first_row", c_void_p), ("seq_slot", c_void_p), ("seq_pos0", c_void_p),
+                ("qkv", c_void_p), ("gates", c_void_p), ("o", c_void_p), ("heads", c_int32), ("kv_heads", c_int32), ("D", c_int32), ("V", c_int32),
+                ("taps", c_int32), ("n_rows", c_int32)]
+
+
+class AddNormArg(Structure):
+    """Mirror of `struct LnArgs` in layer_norm.cu."""
+    _fields_ = [("resid", c_void_p), ("delta", c_void_p), ("bias_d", c_void_p), ("w_d", c_void_p), ("w", c_void_p), ("rows", c_void_p),
+                ("eps_d", c_float), ("eps", c_float), ("centred_d", c_int32), ("centred", c_int32), ("hidden", c_int32)]
+
+
+class LatentTurnArg(Structure):
+    """Mirror of `struct LatentTurn` in mixer_rows.cu."""
+    _fields_ = [("freq", c_void_p), ("table", c_void_p), ("mag", c_float), ("table_positions", c_int32), ("rot", c_int32), ("half_layout", c_int32)]
+
+
+class LatentRowsArg(Structure):
+    """Mirror of `struct LatentRowsArgs` in mixer_rows.cu."""
+    _fields_ = [("src", c_void_p), ("ld", c_int64), ("dq_col", c_int32), ("q_rank", c_int32), ("dkv_col", c_int32), ("rank", c_int32),
+                ("norm_q", c_void_p), ("norm_kv", c_void_p), ("eps", c_float), ("turn", LatentTurnArg), ("row_slot", c_void_p),
+                ("row_pos", c_void_p), ("n_rows", c_int32), ("write_cache", c_int32)]
+
+
 class SampleIOArg(Structure):
     """Mirror of `struct SampleIO` in sampling.cu."""
     _fields_ = [("logits", c_void_p), ("temperature", c_void_p), ("top_p", c_void_p), ("seed", c_void_p),
@@ -164,7 +192,19 @@ _SIGNATURES = {
     "x0ne_whole_norm_rope_kv_write": [_P, _I, _I, _I, _I, _P, _P, _F, _P, _I, _P, _I, _P, _I, None, _P, _P, _I, _I, _P],
     "x0ne_relu2": [_P, _P, _I, _L, _P],
     "x0ne_moe_route": [_P, _I, _P, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P],
-    "x0ne_rope_pairs_kv_write": [_P, _I, _I, _I, _I, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, None, _P, _P, _I, _I, _P],
+    "x0ne_rope_pairs_kv_write": [_P, _P, _I, _I, _I, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _I, _I, None, _P, _P, _I, _I, _P],
+    "x0ne_latent_rows": [LatentRowsArg, _P, _I, None, _P],
+    "x0ne_latent_queries": [_P, _L, _P, _L, LatentTurnArg, _P, _P, _I, _I, _I, _I, _I, _P],
+    "x0ne_heads_gate": [_P, _L, _P, _L, _P, _I, _I, _I, _I, _P],
+    "x0ne_soft_cap": [_P, _L, _F, _P],
+    "x0ne_add_norm": [AddNormArg, _P, _I, _I, _P],
+    "x0ne_delta_prepare": [DeltaArg, _P],
+    "x0ne_delta_scan": [DeltaArg, _I, _P],
+    "x0ne_delta_head_norm": [DeltaArg, _P, _I, _L, _P],
+    "x0ne_delta_step": [DeltaArg, _P, _I, _L, _I, _P],
+    "x0ne_gemm_bf16_smallm_act": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P],
+    "x0ne_gemm_bf16_tcgen05_act": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _I, _F, _P],
+    "x0ne_gemm_bf16_skinny_tcgen05_act": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _P, _I, _F, _P],
     "x0ne_diff_heads": [_P, _P, _L, _P, _I, _I, _I, _I, _F, _F, _F, _P],
     "x0ne_causal_conv_silu": [_P, _L, _I, _P, _P, _P, _L, _L, _P, _P, _P, _I, _I, _I, _P],
     "x0ne_selective_scan": ["ssm", _I, _I, _I, _P],
@@ -1002,9 +1042,20 @@ def gemm_smallm_takes(w: torch.Tensor, m: int, swiglu: bool = False) -> bool:
     return w.dtype == torch.bfloat16 and 0 < m <= SMALL_M_MAX_ROWS and w.shape[1] % 8 == 0 and not (swiglu and w.shape[0] % 2)
 
 
+OUT_RELU2, OUT_SOFT_CAP = 1, 2          # what a plain product's epilogue may do to its result (common.cuh: X0NE_OUT_*)
+
+
+def _out_act(act: tuple, swiglu: bool) -> tuple:
+    """(kind, parameter) of a plain product's activation, checked."""
+    if swiglu or act[0] not in (OUT_RELU2, OUT_SOFT_CAP) or (act[0] == OUT_SOFT_CAP and not act[1] > 0):
+        raise KernelError(f"no product has the activation {act!r} (gated: {swiglu})")
+    return int(act[0]), float(act[1])
+
+
 def gemm_bf16_smallm(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, swiglu: bool = False,
-                     glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None) -> None:
-    """y[:m] = x[:m] @ w.T for m <= 32 by streaming w once; y is bfloat16 or float32.  With
+                     glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None, act: Optional[tuple] = None) -> None:
+    """y[:m] = x[:m] @ w.T for m <= 32 by streaming w once; y is bfloat16 or float32.  `act` = (kind, parameter): the
+    results pass an activation in the epilogue (OUT_RELU2: max(y, 0)^2; OUT_SOFT_CAP: p tanh(y / p)).  With
     `swiglu`, w is the packed [gate; up] weight and y[:m] = silu(x gate^T) * (x up^T); with `glu` =
     (limit, slope, shift) besides, the clipped unit min(g, limit) sigmoid(slope g) (clamp(u) + shift)."""
     lib = _lib("fast")
@@ -1021,6 +1072,10 @@ def gemm_bf16_smallm(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, 
         kind = 2 if swiglu else 0
     else:
         raise KernelError(f"gemm_smallm: no output kind for {y.dtype} (swiglu={swiglu})")
+    if act is not None:
+        a, p = _out_act(act, swiglu)
+        _check(lib, lib.x0ne_gemm_bf16_smallm_act(_ptr(w), _ptr(x), _ptr(y), m, n, k, n, kind, _sms(w.device), a, p, _stream()), "gemm_bf16_smallm")
+        return
     glu = _glu_of(glu, bias, n, swiglu)
     if glu is not None and swiglu:
         _check(lib, lib.x0ne_gemm_bf16_smallm_glu(_ptr(w), _ptr(x), _ptr(y), m, n, k, n, kind, _sms(w.device),
@@ -1073,8 +1128,8 @@ def gemm_tc_status(device) -> torch.Tensor:
 
 
 def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, swiglu: bool = False,
-                      pair: bool = True, glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None) -> None:
-    """y[:m] = x[:m] @ w.T on the tcgen05 tensor cores (128 x 256 tiles, TMA loads, accumulator in
+                      pair: bool = True, glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None, act: Optional[tuple] = None) -> None:
+    """y[:m] = x[:m] @ w.T on the tcgen05 tensor cores, with `act` as for gemm_bf16_smallm (128 x 256 tiles, TMA loads, accumulator in
     tensor memory; with `pair`, pairs of blocks on 256 x 256 tiles); y is bfloat16 or float32.  With `swiglu`, w is the packed [gate; up] weight and
     y[:m] = silu(x gate^T) * (x up^T).  Needs K % 8 == 0."""
     lib = _lib("tc")
@@ -1093,6 +1148,11 @@ def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int,
         raise KernelError(f"gemm_tc: no output kind for {y.dtype} (swiglu={swiglu})")
     global tc_used
     tc_used = True
+    if act is not None:
+        a, p = _out_act(act, swiglu)
+        _check(lib, lib.x0ne_gemm_bf16_tcgen05_act(_ptr(w), _ptr(x), _ptr(y), m, n, k, n, kind, 1 if pair else 0, _ptr(gemm_tc_status(w.device)), a, p,
+                                                   _stream()), "gemm_bf16_tcgen05")
+        return
     glu = _glu_of(glu, bias, n, swiglu)
     if glu is not None and swiglu:       # (limit, slope, shift): the clipped gated unit instead of SwiGLU
         _check(lib, lib.x0ne_gemm_bf16_tcgen05_glu(_ptr(w), _ptr(x), _ptr(y), m, n, k, n, kind, 1 if pair else 0,
@@ -1113,19 +1173,20 @@ def gemm_skinny_tc_takes(w: torch.Tensor, m: int) -> bool:
     return w.dtype == torch.bfloat16 and SKINNY_MIN_ROWS <= m <= SKINNY_MAX_ROWS and w.shape[1] % 8 == 0
 
 
-def product_kernel(w: torch.Tensor, m: int, fused: bool = False) -> str:
+def product_kernel(w: torch.Tensor, m: int, fused: bool = False, act: bool = False) -> str:
     """The kernel the routing table names for m rows against w, or "library" where that kernel does not
-    take the shape (a width that is no multiple of 8)."""
+    take the shape (a width that is no multiple of 8).  `act`: the results pass an activation, which a library product leaves
+    to a launch of its own."""
     from . import routes
-    kernel = routes.kernel_for(m, w.shape[0], w.shape[1], fused=fused, sms=_sms(w.device))
+    kernel = routes.kernel_for(m, w.shape[0], w.shape[1], fused=fused, act=act, sms=_sms(w.device))
     can = {"smallm": gemm_smallm_takes(w, m, fused), "skinny": gemm_skinny_tc_takes(w, m), "tc_pair": gemm_tc_takes(w, m),
            "library": True}[kernel]
     return kernel if can else "library"
 
 
 def gemm_bf16_skinny_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, m: int, swiglu: bool = False,
-                             glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None) -> None:
-    """y[:m] = x[:m] @ w.T for up to 64 rows on tcgen05, K cut over the blocks of a cluster that add
+                             glu: Optional[tuple] = None, bias: Optional[torch.Tensor] = None, act: Optional[tuple] = None) -> None:
+    """y[:m] = x[:m] @ w.T for up to 64 rows on tcgen05 (with `act` as for gemm_bf16_smallm), K cut over the blocks of a cluster that add
     their partial sums through shared memory; y is bfloat16 or float32.  With `swiglu`, w is the
     packed [gate; up] weight and y[:m] = silu(x gate^T) * (x up^T).  Failures of its bounded waits
     show in `gemm_tc_status`."""
@@ -1146,6 +1207,11 @@ def gemm_bf16_skinny_tcgen05(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, 
         raise KernelError(f"gemm_skinny_tc: no output kind for {y.dtype} (swiglu={swiglu})")
     tc_used = True
     x_rows = x.numel() // k      # rows really behind x: the copies may read them all (their results are not used)
+    if act is not None:
+        a, p = _out_act(act, swiglu)
+        _check(lib, lib.x0ne_gemm_bf16_skinny_tcgen05_act(_ptr(w), _ptr(x), x_rows, _ptr(y), m, n, k, n, kind, _ptr(gemm_tc_status(x.device)), a, p,
+                                                          _stream()), "gemm_bf16_skinny_tcgen05")
+        return
     glu = _glu_of(glu, bias, n, swiglu)
     if glu is not None and swiglu:       # (limit, slope, shift): the clipped gated unit instead of SwiGLU
         _check(lib, lib.x0ne_gemm_bf16_skinny_tcgen05_glu(_ptr(w), _ptr(x), x_rows, _ptr(y), m, n, k, n, kind,
@@ -1323,10 +1389,12 @@ def tanh_rows(x: torch.Tensor, out: torch.Tensor, n_rows: int) -> None:
 
 def rope_pairs_kv_write(src: torch.Tensor, k_col: int, v_col: int, freq: Optional[torch.Tensor], table: Optional[torch.Tensor], rot: int,
                         maps: int, dim: int, unit_eps: Optional[float], q_out: torch.Tensor, q_heads: int, q_padded: bool,
-                        cache: PagedCacheArg, row_slot: torch.Tensor, row_pos: torch.Tensor, n_rows: int, write_kv: bool = True) -> None:
-    """Queries (columns from 0), keys (from k_col) and values (from v_col) of the packed projection `src`: of every
-    (head, map) of `dim` values the first `rot` turn as interleaved pairs by pos * freq[i] (`table`: float32
-    [positions, rot], cosines then sines), then, with `unit_eps` not None, it is divided by its root mean square; queries
+                        cache: PagedCacheArg, row_slot: torch.Tensor, row_pos: torch.Tensor, n_rows: int, write_kv: bool = True,
+                        bias: Optional[torch.Tensor] = None, mag: float = 1.0) -> None:
+    """Queries (columns from 0), keys (from k_col) and values (from v_col) of the packed projection `src`, `bias` (float32, one
+    value per column) added to all three: of every (head, map) of `dim` values the first `rot` turn as interleaved pairs by
+    pos * freq[i] (`table`: float32 [positions, rot], cosines then sines; where they are computed they are multiplied by
+    `mag`), then, with `unit_eps` not None, it is divided by its root mean square; queries
     to q_out ([rows, q_heads * maps, dim], or with `q_padded` [rows, q_heads * maps, maps * dim] with zeros beside the
     query's own map), keys (a kv head's maps side by side) and values to the pages."""
     lib = _lib("core")
@@ -1343,8 +1411,12 @@ def rope_pairs_kv_write(src: torch.Tensor, k_col: int, v_col: int, freq: Optiona
     q_width = q_heads * maps * (maps * dim if q_padded else dim)
     if src.numel() < n_rows * src.shape[-1] or q_out.shape[-1] != q_width or q_out.numel() < n_rows * q_width:
         raise KernelError("rope_pairs_kv_write: buffers smaller than the rows asked for")
-    _check(lib, lib.x0ne_rope_pairs_kv_write(_ptr(src), dtype_tag(src.dtype), src.shape[-1], k_col, v_col, _ptr(freq), _ptr(table),
-                                             0 if table is None else table.shape[0], rot, maps, dim,
+    if bias is not None:
+        _need(bias, torch.float32, "projection biases")
+        if bias.numel() != src.shape[-1]:
+            raise KernelError("rope_pairs_kv_write: the biases do not match the projection's columns")
+    _check(lib, lib.x0ne_rope_pairs_kv_write(_ptr(src), _ptr(bias), dtype_tag(src.dtype), src.shape[-1], k_col, v_col, _ptr(freq), _ptr(table),
+                                             0 if table is None else table.shape[0], rot, maps, dim, float(mag),
                                              -1.0 if unit_eps is None else float(unit_eps), _ptr(q_out), q_heads, 1 if q_padded else 0,
                                              cache, _ptr(row_slot), _ptr(row_pos), n_rows, 1 if write_kv else 0, _stream()),
            "rope_pairs_kv_write")
@@ -1655,3 +1727,185 @@ def scan_head_norm(o: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, out
                       _ptr(gate), gate.stride(0) if gate is not None else 0, float(eps), float(post), out.shape[-1], heads, v_dim)
     _check(lib, lib.x0ne_scan_head_norm(arg, out.data_ptr() + out_col * out.element_size(), dtype_tag(out.dtype), n_rows, _stream()),
            "scan_head_norm")
+
+
+# ---------------------------------------------------------------------------------------------
+# norms that subtract the mean (csrc/layer_norm.cu), gated delta rule (csrc/delta_rule.cu), latent rows, heads' gate (module `core`)
+# ---------------------------------------------------------------------------------------------
+def add_norm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, out: torch.Tensor, n_rows: int, eps: float, centred: bool,
+             rows: Optional[torch.Tensor] = None, delta_weight: Optional[torch.Tensor] = None, delta_eps: float = 0.0, delta_centred: bool = False,
+             delta_bias: Optional[torch.Tensor] = None) -> None:
+    """resid += norm(delta + delta_bias) * delta_weight (no delta_weight: the sum as it is; float32, never rounded); out =
+    norm(resid) * weight.  A centred norm subtracts the mean first (layer norm), the other divides by the root mean square.
+    `rows` gathers source rows."""
+    lib = _lib("core")
+    hidden = weight.numel()
+    _need(resid, torch.float32, "residual")
+    _need(weight, torch.float32, "norm weight")
+    _need(out, out.dtype, "norm output")
+    if delta is not None:
+        _need(delta, out.dtype, "delta")
+        if delta.shape[-1] != hidden:
+            raise KernelError("add_norm: delta width differs from the norm's")
+    for t, what in ((delta_weight, "norm weight of the delta"), (delta_bias, "delta bias")):
+        if t is not None:
+            _need(t, torch.float32, what)
+            if t.numel() != hidden or delta is None:
+                raise KernelError(f"add_norm: the {what} does not match a delta")
+    if rows is not None:
+        _need(rows, torch.int32, "row list")
+        if rows.numel() < n_rows:
+            raise KernelError("add_norm: row list shorter than the rows asked for")
+    elif resid.numel() < n_rows * hidden or (delta is not None and delta.numel() < n_rows * hidden):
+        raise KernelError("add_norm: residual or delta smaller than the rows asked for")
+    if resid.shape[-1] != hidden or out.shape[-1] != hidden or out.numel() < n_rows * hidden:
+        raise KernelError("add_norm: widths differ or output too small")
+    arg = AddNormArg(_ptr(resid), _ptr(delta), _ptr(delta_bias), _ptr(delta_weight), _ptr(weight), _ptr(rows), float(delta_eps), float(eps),
+                     1 if delta_centred else 0, 1 if centred else 0, hidden)
+    _check(lib, lib.x0ne_add_norm(arg, _ptr(out), dtype_tag(out.dtype), n_rows, _stream()), "add_norm")
+
+
+def soft_cap(x: torch.Tensor, n_rows: int, cap: float) -> None:
+    """x[:n_rows] = cap * tanh(x / cap) in place; float32."""
+    lib = _lib("core")
+    _need(x, torch.float32, "capped rows")
+    if x.numel() < n_rows * x.shape[-1]:
+        raise KernelError("soft_cap: fewer rows than asked for")
+    _check(lib, lib.x0ne_soft_cap(_ptr(x), n_rows * x.shape[-1], float(cap), _stream()), "soft_cap")
+
+
+def latent_turn(freq: Optional[torch.Tensor], table: Optional[torch.Tensor], mag: float, rot: int, half_layout: bool) -> LatentTurnArg:
+    """How the rotated parts of a latent attention turn."""
+    if rot:
+        _need(freq, torch.float32, "rotary frequencies")
+        if freq.numel() * 2 != rot:
+            raise KernelError("latent_turn: frequencies are not rot / 2")
+    if table is not None:
+        _need(table, torch.float32, "rotary table")
+        if table.dim() != 2 or table.shape[1] != rot:
+            raise KernelError("latent_turn: the table is not [positions, rot]")
+    return LatentTurnArg(_ptr(freq), _ptr(table), float(mag), 0 if table is None else table.shape[0], rot, 1 if half_layout else 0)
+
+
+def latent_rows(src: torch.Tensor, dq_col: int, q_rank: int, norm_q: Optional[torch.Tensor], cq_out: Optional[torch.Tensor], dkv_col: int, rank: int,
+                norm_kv: torch.Tensor, eps: float, turn: LatentTurnArg, cache: PagedCacheArg, row_slot: torch.Tensor, row_pos: torch.Tensor, n_rows: int,
+                write_cache: bool = True) -> None:
+    """RMS norms of a row's query latent (to cq_out) and key/value latent (into the cache), and the shared key part behind the
+    latter, turned, into the cache (see mixer_rows.cu)."""
+    lib = _lib("core")
+    _need(src, src.dtype, "projection rows")
+    _need(norm_kv, torch.float32, "latent norm weight")
+    _need(row_slot, torch.int32, "row slots")
+    _need(row_pos, torch.int32, "row positions")
+    if q_rank:
+        _need(norm_q, torch.float32, "query latent norm weight")
+        _need(cq_out, src.dtype, "query latents")
+        if norm_q.numel() != q_rank or cq_out.shape[-1] != q_rank or cq_out.numel() < n_rows * q_rank:
+            raise KernelError("latent_rows: the query latents do not match their rank")
+    if norm_kv.numel() != rank or src.numel() < n_rows * src.shape[-1]:
+        raise KernelError("latent_rows: widths or rows do not match")
+    arg = LatentRowsArg(_ptr(src), src.shape[-1], dq_col, q_rank, dkv_col, rank, _ptr(norm_q), _ptr(norm_kv), float(eps), turn, _ptr(row_slot),
+                        _ptr(row_pos), n_rows, 1 if write_cache else 0)
+    _check(lib, lib.x0ne_latent_rows(arg, _ptr(cq_out), dtype_tag(src.dtype), cache, _stream()), "latent_rows")
+
+
+def latent_queries(q: torch.Tensor, q_ld: int, q_abs: torch.Tensor, turn: LatentTurnArg, row_pos: torch.Tensor, q_out: torch.Tensor, heads: int, dim: int,
+                   rank: int, n_rows: int) -> None:
+    """q_out[row, head] = [q_abs[head, row] | turned q[row, head, dim:]]; `q` a buffer whose rows start q_ld values apart."""
+    lib = _lib("core")
+    _need(q_abs, q.dtype, "queries in latent space")
+    _need(q_out, q.dtype, "query output")
+    _need(row_pos, torch.int32, "row positions")
+    if q_abs.dim() != 3 or q_abs.shape[0] != heads or q_abs.shape[2] != rank or q_abs.shape[1] < n_rows:
+        raise KernelError("latent_queries: q_abs is not [heads, rows, rank]")
+    if q_out.shape[-1] != heads * (rank + turn.rot) or q_out.numel() < n_rows * q_out.shape[-1] or q.numel() < (n_rows - 1) * q_ld + heads * (dim + turn.rot):
+        raise KernelError("latent_queries: widths or rows do not match")
+    _check(lib, lib.x0ne_latent_queries(_ptr(q), q_ld, _ptr(q_abs), q_abs.stride(0), turn, _ptr(row_pos), _ptr(q_out), dtype_tag(q.dtype), heads, dim, rank,
+                                        n_rows, _stream()), "latent_queries")
+
+
+def heads_gate(x: torch.Tensor, gate: torch.Tensor, gate_ld: int, out: torch.Tensor, n_rows: int) -> None:
+    """out[row, h * V + d] = x[h, row, d] * sigmoid(gate[row, h * V + d]); x [heads, rows, V]; `gate`: a view whose rows start
+    gate_ld values apart."""
+    lib = _lib("core")
+    _need(x, out.dtype, "heads")
+    _need(out, out.dtype, "gated heads")
+    if x.dim() != 3 or x.shape[1] < n_rows or out.shape[-1] != x.shape[0] * x.shape[2] or out.numel() < n_rows * out.shape[-1] or gate.dtype != out.dtype or not gate.is_cuda:
+        raise KernelError("heads_gate: shapes or types do not match")
+    _check(lib, lib.x0ne_heads_gate(_ptr(x), x.stride(0), _ptr(gate), gate_ld, _ptr(out), dtype_tag(out.dtype), n_rows, x.shape[0], x.shape[2], _stream()),
+           "heads_gate")
+
+
+DELTA_STEP_MAX_DIM, DELTA_STEP_MAX_VALUES, DELTA_MAX_TAPS = 256, 2048, 64
+
+
+class DeltaState:
+    """Where the parts of a delta rule's state row lie, and the widths of its heads: `heads` value heads of `v_dim` share
+    `kv_heads` query/key heads of `dim`; convolutions of `taps` taps."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, v_dim: int, taps: int):
+        self.heads, self.kv_heads, self.dim, self.v_dim, self.taps = heads, kv_heads, dim, v_dim, taps
+        if heads % kv_heads or not 1 <= taps <= DELTA_MAX_TAPS:
+            raise ValueError(f"a delta rule of {heads} heads over {kv_heads}, {taps} taps (at most {DELTA_MAX_TAPS})")
+        self.channels = 2 * kv_heads * dim + heads * v_dim
+        self.ring_off = -(-heads * v_dim * dim // 4) * 4
+        self.floats = -(-(self.ring_off + (taps * self.channels if taps > 1 else 0)) // 4) * 4          # (rows of 16 bytes)
+
+    def step_takes(self) -> bool:
+        """Whether the one-launch kernel for passes of one token per sequence takes these widths."""
+        return self.dim <= DELTA_STEP_MAX_DIM and self.v_dim <= DELTA_STEP_MAX_VALUES
+
+
+def delta_arg(g: DeltaState, src: torch.Tensor, cols, conv: torch.Tensor, A: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor, q_scale: float,
+              eps: float, state: torch.Tensor, row_slot: torch.Tensor, row_pos: torch.Tensor, seq_first_row: torch.Tensor, seq_slot: torch.Tensor,
+              seq_pos0: torch.Tensor, n_rows: int, qkv: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None,
+              o: Optional[torch.Tensor] = None) -> DeltaArg:
+    """What the delta rule's kernels read and write.  `src`: the float32 projection; `cols`: where q, k, v, a, b and the output
+    gate start in its rows; `conv` [channels, taps]: q's channels, k's, v's; qkv, gates, o: buffers for passes of many tokens."""
+    for t, what in ((src, "projection"), (conv, "convolution taps"), (A, "decay rates"), (dt_bias, "decay biases"), (norm_w, "head norm weight"), (state, "state"),
+                    (qkv, "prepared rows"), (gates, "gates"), (o, "scan output")):
+        if t is not None:
+            _need(t, torch.float32, what)
+    hv = g.heads * g.v_dim
+    ends = [c + n for c, n in zip(cols, (g.kv_heads * g.dim, g.kv_heads * g.dim, hv, g.heads, g.heads, hv))]
+    if max(ends) > src.shape[-1] or src.numel() < n_rows * src.shape[-1] or tuple(conv.shape) != (g.channels, g.taps) or A.numel() != g.heads \
+            or dt_bias.numel() != g.heads or norm_w.numel() != g.v_dim or state.dim() != 2 or state.shape[1] < g.floats:
+        raise KernelError("delta rule: shapes do not match")
+    for t, width in ((qkv, g.channels), (gates, 2 * g.heads), (o, hv)):
+        if t is not None and (t.shape[-1] != width or t.numel() < n_rows * width):
+            raise KernelError("delta rule: a buffer does not match the heads or rows")
+    return DeltaArg(_ptr(src), src.shape[-1], *cols, _ptr(conv), _ptr(A), _ptr(dt_bias), _ptr(norm_w), float(q_scale), float(eps), _ptr(state), state.stride(0),
+                    g.ring_off, _ptr(row_slot), _ptr(row_pos), _ptr(seq_first_row), _ptr(seq_slot), _ptr(seq_pos0), _ptr(qkv), _ptr(gates), _ptr(o), g.heads,
+                    g.kv_heads, g.dim, g.v_dim, g.taps, n_rows)
+
+
+def delta_prepare(a: DeltaArg) -> None:
+    """Convolution, activation and unit vectors of every row's q, k and v into qkv, decays and write strengths into gates."""
+    lib = _lib("core")
+    _check(lib, lib.x0ne_delta_prepare(a, _stream()), "delta_prepare")
+
+
+def delta_scan(a: DeltaArg, n_seqs: int) -> None:
+    """Token by token over every sequence's prepared rows, from and into its state; the convolutions' inputs join the state."""
+    lib = _lib("core")
+    _check(lib, lib.x0ne_delta_scan(a, n_seqs, _stream()), "delta_scan")
+
+
+def _delta_out(a: DeltaArg, out: torch.Tensor) -> None:
+    _need(out, out.dtype, "gated heads")
+    if out.shape[-1] != a.heads * a.V or out.numel() < a.n_rows * out.shape[-1]:
+        raise KernelError("delta rule: the output does not match the heads or rows")
+
+
+def delta_head_norm(a: DeltaArg, out: torch.Tensor) -> None:
+    """out = o / sqrt(mean(o^2) + eps) * weight * silu(gate) per head."""
+    lib = _lib("core")
+    _delta_out(a, out)
+    _check(lib, lib.x0ne_delta_head_norm(a, _ptr(out), dtype_tag(out.dtype), out.shape[-1], _stream()), "delta_head_norm")
+
+
+def delta_step(a: DeltaArg, out: torch.Tensor, n_seqs: int) -> None:
+    """All of it in one launch where every sequence brings one row: the bits of the three kernels above."""
+    lib = _lib("core")
+    _delta_out(a, out)
+    _check(lib, lib.x0ne_delta_step(a, _ptr(out), dtype_tag(out.dtype), out.shape[-1], n_seqs, _stream()), "delta_step")

@@ -54,6 +54,7 @@ class Rule:
     fused: Optional[bool]                       # True: gate|up with the SwiGLU epilogue only; False: plain only; None: both
     when: Callable[[Shape], bool]
     why: str
+    act: Optional[bool] = None                  # True: plain products whose results pass an activation only; None: both
 
 
 def _always(s: Shape) -> bool:
@@ -100,14 +101,15 @@ RULES: List[Rule] = [
 ]
 
 
-def choose(rows: int, n: int, k: int, *, fused: bool = False, sms: int = 148) -> Rule:
-    """The first rule that covers `rows` rows of x against W [n, k] (n = 2 x intermediate when `fused`)."""
+def choose(rows: int, n: int, k: int, *, fused: bool = False, act: bool = False, sms: int = 148) -> Rule:
+    """The first rule that covers `rows` rows of x against W [n, k] (n = 2 x intermediate when `fused`; `act`: a plain
+    product whose results pass an activation)."""
     s = Shape(n, k, sms)
     for r in RULES:
-        if r.rows[0] <= rows <= r.rows[1] and (r.fused is None or r.fused == fused) and r.when(s):
+        if r.rows[0] <= rows <= r.rows[1] and (r.fused is None or r.fused == fused) and (r.act is None or r.act == act) and r.when(s):
             return r
     raise ValueError(f"no rule for {rows} rows of a {n} x {k} product")     # the last rule matches everything
 
 
-def kernel_for(rows: int, n: int, k: int, *, fused: bool = False, sms: int = 148) -> str:
-    return choose(rows, n, k, fused=fused, sms=sms).kernel
+def kernel_for(rows: int, n: int, k: int, *, fused: bool = False, act: bool = False, sms: int = 148) -> str:
+    return choose(rows, n, k, fused=fused, act=act, sms=sms).kernel

@@ -108,6 +108,9 @@ class Norm(Part):
 
 
 class Mixer(Part):
+    defer_bias = False          # True: the arrangement adds `result_bias` (if there is one) itself, where it adds the result
+    result_bias: Optional[torch.Tensor] = None
+
     @staticmethod
     def cache_need(spec: PartSpec) -> CacheNeed:
         return CacheNeed()

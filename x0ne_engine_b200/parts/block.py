@@ -58,7 +58,7 @@ class SandwichBlock(Block):
     after it, on its result, before the add.  The normed result is never stored: the result travels with its
     norm (`PostNormed`) to the next norm in line, whose kernel norms it, adds it to the float32 residual
     and norms the sum.  A layer may leave the feed-forward (and its two norms) out.  With `mixer_input` an input transform
-    stands between the first norm and the mixer.  A feed-forward's result bias travels with its result."""
+    stands between the first norm and the mixer.  A mixer's or feed-forward's result bias travels with its result."""
     replayable = True
     ROLES = {"mixer_norm": "norm", "mixer_input": "input_transform", "mixer": "mixer", "mixer_post_norm": "norm", "ffn_norm": "norm",
              "ffn": "feed_forward", "ffn_post_norm": "norm"}
@@ -68,6 +68,7 @@ class SandwichBlock(Block):
         super().__init__(parts)
         if (self.ffn is None) != (self.ffn_norm is None) or (self.ffn is None) != (self.ffn_post_norm is None):
             raise ValueError("a sandwich layer has its feed-forward with both of its norms, or none of the three")
+        self.mixer.defer_bias = True
         if self.ffn is not None:
             self.ffn.defer_bias = True
 
@@ -79,7 +80,7 @@ class SandwichBlock(Block):
             self.mixer_norm.add_norm(ctx, resid, delta, normed, ctx.n_rows)
             read = normed
         mixed = PostNormed(self.mixer.forward(ctx, entry, read, ctx.n_rows, cache_entry=cache_entry, write_cache=write_cache),
-                           self.mixer_post_norm)
+                           self.mixer_post_norm, self.mixer.result_bias)
         if self.ffn is None:
             return mixed
         self.ffn_norm.add_norm(ctx, resid, mixed, normed, ctx.n_rows)

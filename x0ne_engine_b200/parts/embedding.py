@@ -114,8 +114,8 @@ class ConcatOpener(Opener):
             norm, bias, delta = delta.norm, delta.bias, delta.delta
         elif delta is not None and not isinstance(delta, torch.Tensor):
             raise ValueError("a concatenating opener takes the pending result of a layer as one tensor")
-        if norm is not None and norm.groups != 1:
-            raise ValueError("a norm in groups does not take a result that is still to be normed")
+        if norm is not None and (norm.groups != 1 or norm.centred):
+            raise ValueError("a concatenating opener takes a result that is still to be normed by one root mean square only")
         x0 = ws.buffer(EMBEDDING_OUTPUT, (ws.max_rows, h), torch.float32)
         cat = ws.buffer("opener.rows", (ws.max_rows, 2 * h), dt)
         ops.concat_rows(resid, delta, bias, None if norm is None else norm.weight, 0.0 if norm is None else norm.eps, x0, cat, n_rows)
@@ -162,13 +162,14 @@ class PassOpener(Opener):
 
 class LMHead(Head):
     """logits = normed W^T in float32 for the wanted rows only; W is the embedding table when the
-    model is tied (x0ne-core/runtime/src/engine.rs:823-835).  Parameters: vocab_size,
-    hidden_size, tied, names.weight."""
+    model is tied (x0ne-core/runtime/src/engine.rs:823-835).  With `softcap` they become softcap * tanh(logits / softcap).
+    Parameters: vocab_size, hidden_size, tied, softcap (default: none), names.weight."""
     replayable = True
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
         self.linear = None
+        self.act = (ops.OUT_SOFT_CAP, float(spec["softcap"])) if spec.get("softcap") else None
 
     @staticmethod
     def tensor_needs(spec: PartSpec) -> List[TensorNeed]:
@@ -187,7 +188,7 @@ class LMHead(Head):
         return self.linear.weight_bytes()
 
     def forward(self, normed, logits, n_rows):
-        return self.linear(normed, logits, n_rows)
+        return self.linear(normed, logits, n_rows, act=self.act)
 
 
 EMBEDDINGS.register("token_embedding", TokenEmbedding)

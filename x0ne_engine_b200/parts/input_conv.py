@@ -56,7 +56,7 @@ class CausalInputConv(InputTransform):
 
     def _fuses(self, norm, delta) -> bool:
         return type(norm) is RMSNorm and norm.groups == 1 and ops.norm_conv_step_takes(self.hidden) and \
-            (delta is None or isinstance(delta, PostNormed) and delta.norm.groups == 1)
+            (delta is None or isinstance(delta, PostNormed) and delta.norm.groups == 1 and not delta.norm.centred)
 
 
 INPUT_TRANSFORMS.register("causal_input_conv", CausalInputConv)

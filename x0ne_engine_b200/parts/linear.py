@@ -7,6 +7,8 @@ library engine delegates these products to cuBLAS (x0ne-core/runtime/src/gpu.rs:
 """
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from ..csrc import ops
@@ -22,12 +24,14 @@ class Linear:
     def weight_bytes(self) -> int:
         return self.weight.numel() * self.weight.element_size()
 
-    def __call__(self, x: torch.Tensor, out: torch.Tensor, m: int) -> torch.Tensor:
-        """out[:m] = x[:m] @ W^T.  `out` has the dtype of x, or float32 (logits)."""
+    def __call__(self, x: torch.Tensor, out: torch.Tensor, m: int, act: Optional[tuple] = None) -> torch.Tensor:
+        """out[:m] = x[:m] @ W^T.  `out` has the dtype of x, or float32 (logits).  `act` = (kind, parameter): what becomes of the
+        results before they are stored (`ops.OUT_RELU2`; `ops.OUT_SOFT_CAP` for float32 results), in the product's epilogue
+        where one of this library's kernels takes the shape."""
         w = self.weight
         if w.dtype == torch.float32:
             ops.gemm_f32_nt(x, w, out, m)
-            return out
+            return self._behind(out, m, act)
         if w.dtype != torch.bfloat16:
             raise ops.KernelError(f"no matrix product for weights of {w.dtype}")
         if out.dtype == torch.float32:
@@ -36,14 +40,29 @@ class Linear:
             # 203 us at 12 rows)
             kernel = "smallm" if m <= 8 and ops.gemm_smallm_takes(w, m) else "library"
         else:
-            kernel = ops.product_kernel(w, m)          # the routing table (csrc/routes.py)
+            kernel = ops.product_kernel(w, m, act=act is not None)          # the routing table (csrc/routes.py)
         if kernel == "smallm":
-            ops.gemm_bf16_smallm(x, w, out, m)
+            ops.gemm_bf16_smallm(x, w, out, m, act=act)
         elif kernel == "skinny":
-            ops.gemm_bf16_skinny_tcgen05(x, w, out, m)
+            ops.gemm_bf16_skinny_tcgen05(x, w, out, m, act=act)
+        elif kernel == "tc_pair":
+            ops.gemm_bf16_tcgen05(x, w, out, m, act=act)
         elif m > 0:
             if out.dtype == torch.bfloat16:
                 torch.mm(x[:m], w.t(), out=out[:m])
             else:
                 torch.mm(x[:m], w.t(), out_dtype=torch.float32, out=out[:m])
+            self._behind(out, m, act)
+        return out
+
+    @staticmethod
+    def _behind(out: torch.Tensor, m: int, act: Optional[tuple]) -> torch.Tensor:
+        """The activation in a launch of its own, behind a product whose epilogue has none."""
+        if act is not None and m > 0:
+            if act[0] == ops.OUT_RELU2:
+                ops.relu2(out, out, m)
+            elif act[0] == ops.OUT_SOFT_CAP:
+                ops.soft_cap(out, m, act[1])
+            else:
+                raise ops.KernelError(f"no activation {act!r}")
         return out

@@ -1,4 +1,4 @@
-"""Dense feed-forwards: SiLU-gated units, and a two-product unit with biases."""
+"""Dense feed-forwards: SiLU-gated units, two products with biases, two products around a squared ReLU."""
 from __future__ import annotations
 
 import math
@@ -154,6 +154,39 @@ class BiasedMLP(FeedForward):
         return out
 
 
+class SquaredReluMLP(FeedForward):
+    """down(max(up x, 0)^2): two products without gate or biases; the activation is in the first product's epilogue wherever one
+    of this library's kernels runs it.
+    Parameters: hidden_size, intermediate_size, names.{up, down}."""
+    replayable = True
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.hidden = int(spec["hidden_size"])
+        self.inter = int(spec["intermediate_size"])
+        self.up = self.down = None
+
+    @staticmethod
+    def tensor_needs(spec: PartSpec) -> List[TensorNeed]:
+        h, i, n = int(spec["hidden_size"]), int(spec["intermediate_size"]), spec["names"]
+        return [TensorNeed(n["up"], (i, h)), TensorNeed(n["down"], (h, i))]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        n = self.spec["names"]
+        self.up, self.down = Linear(tensors[n["up"]]), Linear(tensors[n["down"]])
+
+    def weight_bytes(self) -> int:
+        return self.up.weight_bytes() + self.down.weight_bytes()
+
+    def forward(self, ctx, x, n_rows):
+        z = ctx.ws.buffer("ffn.act", (ctx.ws.max_rows, self.inter), self.env.dtype)
+        out = ctx.ws.buffer(self.out_buffer, (ctx.ws.max_rows, self.hidden), self.env.dtype)
+        self.up(x, z, n_rows, act=(ops.OUT_RELU2, 0.0))
+        self.down(z, out, n_rows)
+        return out
+
+
 FEED_FORWARDS.register("swiglu", SwiGLU)
+FEED_FORWARDS.register("squared_relu_mlp", SquaredReluMLP)
 FEED_FORWARDS.register("biased_mlp", BiasedMLP)
 FEED_FORWARDS.register("clipped_glu", ClippedGLU)
