@@ -13,9 +13,9 @@ time); `e2e` is the same rate through `Model.generate` with host token lists in 
 and 64 and the milliseconds a 128-token and a 512-token prompt take through the step function; `roofline` places the decode step against the bytes it must read.  One JSON line is
 printed.  This library runs on one GPU: for --gpus above 1 a line says so and the exit code is 2.
 
-    python bench.py --design rovurax|tenetar|retuvik|barorax|ravapel [--sizes 1.7b,8b] [--layers 8] [--chunk 1024] [--steps K]
+    python bench.py --design rovurax|tenetar|retuvik|barorax|ravapel|tarudra [--sizes 1.7b,8b] [--layers 8] [--chunk 1024] [--steps K]
 
-instead runs that design beside Qwen3 (retuvik: beside Tenetar; barorax and ravapel: beside Retuvik) at equal sizes (random bfloat16 weights, the same engine,
+instead runs that design beside Qwen3 (retuvik: beside Tenetar; barorax and ravapel: beside Retuvik; tarudra: beside Ravapel) at equal sizes (random bfloat16 weights, the same engine,
 step function and decode graphs): one prompt of --prefill-tokens through the step function, then decode
 at --batch, device-timed; one JSON line with a row per size and design.
 """
@@ -235,6 +235,28 @@ def ravapel_config(size: dict, layers: int, vocab: int, chunk: int):
                              "loop": {"start": 0, "stop": layers, "times": 1}})
 
 
+def tarudra_config(size: dict, layers: int, vocab: int, window: int):
+    """A Tarudra configuration of the given layer sizes.  Every other layer is the gated delta rule (heads of 128 x 128 that fill the
+    width, half as many query/key heads, 4 taps); of the rest every second is windowed attention with YaRN-scaled rotation, of
+    which the odd ones read the keys and values of the one before, and every second latent attention (the size's latent and
+    rotated part, query latents of a quarter of the width) over the same window; every layer has the dense squared-ReLU
+    feed-forward of one and a half times the size's width, which makes it as many products per token as a gated unit."""
+    from x0ne_engine_b200.config import config_from_dict
+    w, ff, H, G, d = size["width"], size["ff"], size["heads"], size["kv_heads"], size["dim"]
+    rec = {"type": "delta", "mixer": {"conv": 4, "dim": 128, "heads": w // 128, "kv_heads": w // 256, "vdim": 128}}
+    rot = {"base": 1000000.0, "dims": d, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    lat = {"type": "latent_attention", "mixer": {"dim": d, "heads": H, "kv_rank": size["kv_rank"], "q_rank": w // 4, "rot_dim": size["rot_dim"], "vdim": d,
+                                                 "scale": (d + size["rot_dim"]) ** -0.5, "mask": {"size": window},
+                                                 "rot": {"base": 1000000.0, "dims": size["rot_dim"]}}}
+    out = []
+    for i in range(layers):
+        att = {"type": "attention", "mixer": {"dim": d, "heads": H, "kv_heads": G, "vdim": d, "scale": d ** -0.5, "mask": {"size": window}, "rot": rot}}
+        if i % 8 == 5:
+            att["mixer"]["kv_from"] = i - 4
+        out.append({**(rec if i % 2 == 0 else att if i % 4 == 1 else lat), "mlp": {"kind": "dense", "ff": ff * 3 // 2}})
+    return config_from_dict({"architecture": "Tarudra", "vocab": vocab, "width": w, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "layers": out})
+
+
 def design_configs(size: dict, layers: int, vocab: int, chunk: int, design: str = "rovurax"):
     """(the design's configuration, Qwen3 configuration) with the same width, heads, feed-forward, depth and
     vocabulary.  Of every four Rovurax layers three are chunk-masked attention with blended values and
@@ -253,6 +275,8 @@ def design_configs(size: dict, layers: int, vocab: int, chunk: int, design: str 
         return barorax_config(size, layers, vocab, chunk), retuvik_config(size, layers, vocab, chunk)
     if design == "ravapel":        # beside Retuvik: matrix states per head, attention over a bounded span, a repeated stretch
         return ravapel_config(size, layers, vocab, chunk), retuvik_config(size, layers, vocab, chunk)
+    if design == "tarudra":        # beside Ravapel: matrix states per head, attention over a bounded span, dense feed-forwards, norms around each sublayer
+        return tarudra_config(size, layers, vocab, chunk), ravapel_config(size, layers, vocab, chunk)
     mlp = {"ff": ff, "kind": "dense", "limit": 7.0}
     att = {"type": "attention", "mlp": mlp, "mixer": {"dim": d, "heads": H, "kv_heads": G, "vdim": d, "scale": d ** -0.5,
                                                         "mask": {"size": chunk}, "v_mix": True}}
@@ -279,7 +303,7 @@ def design_bench(args) -> int:
     layers = args.layers or 8
     vocab = 32768
     rows_out = []
-    other = {"retuvik": "tenetar", "barorax": "retuvik", "ravapel": "retuvik"}.get(args.design, "qwen3")
+    other = {"retuvik": "tenetar", "barorax": "retuvik", "ravapel": "retuvik", "tarudra": "ravapel"}.get(args.design, "qwen3")
     for name in args.sizes.split(","):
         size = DESIGN_SIZES[name]
         for design, cfg in zip((args.design, other), design_configs(size, layers, vocab, args.chunk, args.design)):
@@ -353,12 +377,12 @@ def main() -> int:
     ap.add_argument("--prefill-tokens", type=int, default=2048)
     ap.add_argument("--no-points", action="store_true", help="skip decode at batch 1 and 64")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--design", default=None, choices=["rovurax", "tenetar", "retuvik", "barorax", "ravapel"],
-                    help="instead of the default workload: this design beside Qwen3 (retuvik: beside Tenetar; barorax and ravapel: beside Retuvik) "
+    ap.add_argument("--design", default=None, choices=["rovurax", "tenetar", "retuvik", "barorax", "ravapel", "tarudra"],
+                    help="instead of the default workload: this design beside Qwen3 (retuvik: beside Tenetar; barorax and ravapel: beside Retuvik; tarudra: beside Ravapel) "
                          "at equal sizes (prefill and decode)")
     ap.add_argument("--sizes", default="1.7b,8b", help="with --design: which of " + ", ".join(DESIGN_SIZES))
     ap.add_argument("--chunk", type=int, default=1024,
-                    help="with --design: positions per chunk of the masked attention (rovurax, barorax, ravapel) or of the sliding window (tenetar, retuvik)")
+                    help="with --design: positions per chunk of the masked attention (rovurax, barorax, ravapel) or of the sliding window (tenetar, retuvik, tarudra)")
     args = ap.parse_args()
     if args.design is not None and args.impl == "ours" and args.gpus == 1:
         return design_bench(args)

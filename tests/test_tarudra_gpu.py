@@ -96,8 +96,9 @@ class Delta:
     def rows(self, n):
         return torch.randn(n, self.width, generator=self.gen)
 
-    def run(self, cut, dtype=torch.float32, step=False):
-        """`cut`: (slot, rows) of one pass, slots of -1 being no sequence's; returns the gated heads."""
+    def run(self, cut, dtype=torch.float32, step=False, chunks=False):
+        """`cut`: (slot, rows) of one pass, slots of -1 being no sequence's; returns the gated heads.  `chunks`: by the scan that takes
+        several tokens together."""
         ops, g = self.ops, self.g
         slots, pos0, pos, row_slot = [], [], [], []
         for s, x in cut:
@@ -111,7 +112,7 @@ class Delta:
         src = torch.cat([x for _, x in cut]).to(DEV)
         n, first = src.shape[0], i32(np.concatenate([[0], np.cumsum([x.shape[0] for _, x in cut])]))
         out = torch.full((n, g.heads * g.v_dim), float("nan"), dtype=dtype, device=DEV)
-        many = {} if step else dict(qkv=torch.empty((n, g.channels), device=DEV), gates=torch.empty((n, 2 * g.heads), device=DEV),
+        many = {} if step else dict(planes=torch.full((n, g.plane_floats), float("nan"), device=DEV), gates=torch.empty((n, 4 * g.heads), device=DEV),
                                     o=torch.zeros((n, g.heads * g.v_dim), device=DEV))
         tabs = [i32(row_slot), i32(pos), first, i32(slots), i32(pos0)]
         a = ops.delta_arg(g, src, self.cols, *self.dev, g.dim ** -0.5, self.eps, self.state, *tabs, n, **many)
@@ -119,7 +120,10 @@ class Delta:
             ops.delta_step(a, out, len(slots))
         else:
             ops.delta_prepare(a)
-            ops.delta_scan(a, len(slots))
+            if chunks:
+                ops.delta_chunk_scan(a, torch.full((n, ops.DELTA_COEF * g.heads), float("nan"), device=DEV), len(slots), max(x.shape[0] for _, x in cut))
+            else:
+                ops.delta_scan(a, len(slots))
             ops.delta_head_norm(a, out)
         torch.cuda.synchronize()
         return out
@@ -161,13 +165,16 @@ def close_rows(got, want, what, tol=2e-4):
     assert err.max() <= tol, f"{what}: {float(err.max()):.2e}"
 
 
+@pytest.mark.parametrize("chunks", [False, True])
 @pytest.mark.parametrize("heads,kv,dim,vd,taps", DELTA_SIZES)
-def test_delta_rule_over_unequal_sequences_and_again_from_the_state(heads, kv, dim, vd, taps):
+def test_delta_rule_over_unequal_sequences_and_again_from_the_state(heads, kv, dim, vd, taps, chunks):
+    if chunks and dim > 256:
+        pytest.skip("the scan by chunks takes heads of up to 256 channels")
     d = Delta(heads, kv, dim, vd, taps, seed=dim + taps)
     got = {}
     for cut in ([(3, 1), (0, 40), (4, 33), (-1, 2)], [(3, 2), (0, 1), (1, 25)], [(1, 1), (0, 16), (3, 70)]):
         rows = [(s, d.rows(n)) for s, n in cut]
-        out, at = d.run(rows).double().cpu(), 0
+        out, at = d.run(rows, chunks=chunks).double().cpu(), 0
         for s, x in rows:
             if s >= 0:
                 got.setdefault(s, []).append(out[at:at + x.shape[0]])
@@ -210,7 +217,8 @@ def test_other_cuts_of_the_scan_give_the_same_bits():
         assert torch.equal(torch.cat(got), want) and torch.equal(a.state, b.state), cuts[:3]
 
 
-def test_a_token_read_from_the_state_600_rows_later():
+@pytest.mark.parametrize("chunks", [False, True])
+def test_a_token_read_from_the_state_600_rows_later(chunks):
     """Hardly any decay; token 0 alone writes one direction that no later key touches, and the last query asks for it."""
     d = Delta(1, 1, 32, 16, 1, seed=3, decay=(-14.0, -13.0))
     x = d.rows(601)
@@ -229,7 +237,7 @@ def test_a_token_read_from_the_state_600_rows_later():
         d.seqs.clear()
         at = 0
         for n in cut:
-            out = d.run([(0, x[at:at + n])])
+            out = d.run([(0, x[at:at + n])], chunks=chunks)
             at += n
         want = d.plain(x)[0]
         close_rows(out[-1:].double().cpu(), want[-1:], "far token", 1e-4)
@@ -238,11 +246,24 @@ def test_a_token_read_from_the_state_600_rows_later():
         assert (d.plain(y)[0][-1] - want[-1]).abs().max() > 0.1 * want[-1].abs().max()
 
 
-def test_a_decay_close_to_one_keeps_its_digits():
+@pytest.mark.parametrize("chunks", [False, True])
+def test_a_decay_close_to_one_keeps_its_digits(chunks):
     d = Delta(2, 1, 16, 8, 2, seed=4, decay=(-15.5, -14.0))
     x = d.rows(1000)
-    got = d.run([(0, x)]).double().cpu()
+    got = d.run([(0, x)], chunks=chunks).double().cpu()
     close_rows(got[-50:], d.plain(x)[0][-50:], "1,000 tokens")
+    d.check_states()
+
+
+def test_decays_that_forget_at_once_and_writes_of_full_strength():
+    """Decays down to nothing and write strengths near one inside the chunks: no product of decays may be divided by."""
+    d = Delta(2, 1, 24, 16, 2, seed=5, decay=(2.0, 60.0))
+    d.A.fill_(3.0)
+    d.dev[1].fill_(3.0)
+    x = d.rows(75)
+    x[::7, d.cols[3]:d.cols[3] + 2] -= 80.0                # every seventh token keeps everything
+    x[:, d.cols[4]:d.cols[4] + 2] += 6.0
+    close_rows(d.run([(0, x)], chunks=True).double().cpu(), d.plain(x)[0], "sharp decays")
     d.check_states()
 
 

@@ -608,6 +608,75 @@ def cmd_kernel_bench(a) -> int:
             extra = dict(nq=nq, em=em, tiny=1e-6, gate=v) if hg else {}
             timed(lambda: ops.scan_head_norm(o, weight, act, 0, rows, heads, vd, 1e-6, **extra), rows * hv * (4 + 2 + (4 if hg else 0)))
         return 0
+    if a.kernel in ("delta_prepare", "delta_scan", "delta_chunk_scan", "delta_head_norm", "delta_step"):
+        # the gated delta rule's own kernels: --batch sequences of --m rows each, --q-heads value heads over --kv-heads of --head-dim
+        # channels x --v-dim values, 4 taps; every sequence goes on from its state
+        B, per, heads, kv, d, taps = a.batch, a.m, a.q_heads, a.kv_heads, a.head_dim, 4
+        vd = a.v_dim or d
+        rows, hk, hv = B * per, kv * d, heads * vd
+        g = ops.DeltaState(heads, kv, d, vd, taps)
+        copies = 1
+        cols = [0, hk, 2 * hk, 2 * hk + hv, 2 * hk + hv + heads, 2 * hk + hv + 2 * heads]
+        src = torch.randn(rows, cols[5] + hv, device=dev)
+        conv, state = torch.randn(g.channels, taps, device=dev) * 0.5, torch.zeros(B, g.floats, device=dev)
+        A, dt_bias, norm = torch.rand(heads, device=dev), torch.rand(heads, device=dev) - 4.0, torch.ones(vd, device=dev)
+        i32 = dict(dtype=torch.int32, device=dev)
+        slots, first = torch.arange(B, **i32), (torch.arange(B + 1, **i32) * per).contiguous()
+        row_slot, row_pos, pos0 = slots.repeat_interleave(per).contiguous(), (torch.arange(per, **i32) + 8).repeat(B).contiguous(), torch.full((B,), 8, **i32)
+        planes, gates, o = torch.empty(rows, g.plane_floats, device=dev), torch.empty(rows, 4 * heads, device=dev), torch.empty(rows, hv, device=dev)
+        act = torch.empty(rows, hv, device=dev, dtype=torch.bfloat16)
+        arg = ops.delta_arg(g, src, cols, conv, A, dt_bias, norm, d ** -0.5, 1e-6, state, row_slot, row_pos, first, slots, pos0, rows, planes=planes, gates=gates, o=o)
+        ops.delta_prepare(arg)
+        ops.delta_scan(arg, B)
+        states, flops = 2 * B * heads * vd * d * 4, 8.0 * rows * heads * d * vd
+        if a.kernel == "delta_prepare":
+            timed(lambda: ops.delta_prepare(arg), rows * g.channels * (4 + 4))
+        elif a.kernel == "delta_scan":
+            timed(lambda: ops.delta_scan(arg, B), rows * (g.channels + hv) * 4 + states, flops)
+        elif a.kernel == "delta_chunk_scan":
+            coef = torch.empty(rows, heads * ops.DELTA_COEF, device=dev)
+            timed(lambda: ops.delta_chunk_scan(arg, coef, B, per), rows * (g.channels + hv) * 4 + states, flops)
+        elif a.kernel == "delta_head_norm":
+            timed(lambda: ops.delta_head_norm(arg, act), rows * hv * (4 + 4 + 2))
+        else:
+            if per != 1:
+                raise SystemExit("delta_step takes one row per sequence: --m 1")
+            timed(lambda: ops.delta_step(arg, act, B), rows * (g.channels * (1 + 2 * taps) * 4 + hv * (4 + 2)) + states, flops)
+        return 0
+    if a.kernel in ("add_norm", "heads_gate", "latent_rows", "latent_queries"):
+        # --m rows: the add of a pending result that is layer-normed first and the layer norm of the sum (--n values); the heads of a
+        # product per head gated and laid side by side (--q-heads x --v-dim); latent attention's rows and queries (--latent-rank
+        # latents, query latents of --n, a rotated part of 64)
+        from .cache import SequenceCache
+        from .parts.base import CacheNeed
+        rows, h, heads, d, rank, rot = a.m, a.n, a.q_heads, a.head_dim, a.latent_rank or 256, 64
+        vd = a.v_dim or d
+        copies = 1
+        bf = lambda *s: torch.randn(*s, device=dev).bfloat16()      # noqa: E731
+        if a.kernel == "add_norm":
+            resid, delta, w = torch.randn(rows, h, device=dev), bf(rows, h), torch.ones(h, device=dev)
+            out = torch.empty_like(delta)
+            timed(lambda: ops.add_norm(resid, delta, w, out, rows, 1e-6, True, delta_weight=w, delta_eps=1e-6, delta_centred=True), rows * h * (4 + 4 + 2 + 2))
+            return 0
+        if a.kernel == "heads_gate":
+            x, gate = bf(heads, rows, vd), bf(rows, heads * vd)
+            out = torch.empty_like(gate)
+            timed(lambda: ops.heads_gate(x, gate, heads * vd, out, rows), rows * heads * vd * 6)
+            return 0
+        cache = SequenceCache([CacheNeed("kv", 1, rank + rot, None, v_dim=0)], [None], rows + 64, rows + 64, torch.bfloat16, dev)
+        slot = cache.acquire(rows)
+        freq, table = torch.rand(rot // 2, device=dev), torch.rand(rows, rot, device=dev)
+        turn = ops.latent_turn(freq, table, 1.0, rot, True)
+        slots, pos = torch.full((rows,), slot, dtype=torch.int32, device=dev), torch.arange(rows, dtype=torch.int32, device=dev)
+        if a.kernel == "latent_rows":
+            src, cq = bf(rows, h + rank + rot), torch.empty(rows, h, device=dev, dtype=torch.bfloat16)
+            wq, wkv = torch.ones(h, device=dev), torch.ones(rank, device=dev)
+            timed(lambda: ops.latent_rows(src, 0, h, wq, cq, h, rank, wkv, 1e-6, turn, cache.kv_view(0), slots, pos, rows), rows * (h + rank + rot) * 4)
+            return 0
+        q, q_abs = bf(rows, heads * (d + rot)), bf(heads, rows, rank)
+        out = torch.empty(rows, heads * (rank + rot), device=dev, dtype=torch.bfloat16)
+        timed(lambda: ops.latent_queries(q, heads * (d + rot), q_abs, turn, pos, out, heads, d, rank, rows), rows * heads * (rank + rot) * 4)
+        return 0
     if a.kernel in ("input_conv", "norm_conv_step", "concat_rows", "embed_sum"):
         # --m rows of --n values: the input convolution of one sequence (4 taps); the residual add, norm and convolution of one
         # row per sequence; the concatenating opener's operand; the summed embedding

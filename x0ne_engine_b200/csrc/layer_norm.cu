@@ -5,24 +5,24 @@
 // float32, d is never rounded; the sum of squared deviations is taken around the mean itself.  One block per row.
 #include "common.cuh"
 
-#define LN_MAX_WARPS 32
+#define LN_MAX_WARPS 16
 
-// Sum and sum of squared deviations of a row whose values lie in the threads' registers.  A warp's mean comes first, then its
-// deviations from that; the warps' parts (count, mean, deviations) meet in shared memory, where every thread adds them up in
-// warp order: deviations from the row's mean are those from the warp's plus count times the square of the means' difference.
-// `parts` [LN_MAX_WARPS][3] must not be in use.
+// Mean and mean squared deviation of a row whose values lie in the threads' registers (`count` of a thread's N, `total` in all).
+// A warp's mean comes first, then its deviations from that; the warps' parts (count, mean, deviations) meet in shared memory,
+// where every warp adds them up, one part per lane: deviations from the row's mean are those from the warp's plus count times the
+// square of the means' difference.  `parts` must not be in use.
 struct LnStats {
     float mean, dev2;           // dev2: mean squared deviation from the mean
 };
 template <int N>
-__device__ __forceinline__ LnStats ln_stats(const float (&x)[N], int count, float (*parts)[3], int total) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+__device__ __forceinline__ LnStats ln_stats(const float (&x)[N], int count, int warp_count, float4* parts, int total) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     float s = 0.f;
 #pragma unroll
     for (int i = 0; i < N; ++i)
         if (i < count) s += x[i];
-    const float n = warp_sum((float)count);
-    const float mean_w = n > 0.f ? warp_sum(s) / n : 0.f;
+    const float n = (float)warp_count;
+    const float mean_w = warp_count > 0 ? warp_sum(s) / n : 0.f;
     float d2 = 0.f;
 #pragma unroll
     for (int i = 0; i < N; ++i)
@@ -31,19 +31,11 @@ __device__ __forceinline__ LnStats ln_stats(const float (&x)[N], int count, floa
             d2 = fmaf(d, d, d2);
         }
     d2 = warp_sum(d2);
-    if (lane == 0) {
-        parts[warp][0] = n;
-        parts[warp][1] = mean_w;
-        parts[warp][2] = d2;
-    }
+    if (lane == 0) parts[warp] = make_float4(n, mean_w, d2, 0.f);
     __syncthreads();
-    float sum = 0.f, dev = 0.f;
-    for (int w = 0; w < warps; ++w) sum = fmaf(parts[w][0], parts[w][1], sum);
-    const float mean = sum / (float)total;
-    for (int w = 0; w < warps; ++w) {
-        const float d = parts[w][1] - mean;
-        dev += fmaf(parts[w][0] * d, d, parts[w][2]);
-    }
+    const float4 p = lane < (int)(blockDim.x >> 5) ? parts[lane] : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float mean = warp_sum(p.x * p.y) / (float)total;
+    const float d = p.y - mean, dev = warp_sum(fmaf(p.x * d, d, p.z));
     return {mean, dev / (float)total};
 }
 // what is taken off, and what the rest is multiplied by
@@ -89,19 +81,22 @@ __device__ __forceinline__ void ln_store8(bf16* p, const float* v) {
     *reinterpret_cast<uint4*>(p) = u;
 }
 
-// hidden % 8 == 0, at most 8 values x ITS sweeps per thread, 16-byte aligned rows: row and delta stay in registers, weights are
-// asked for before the wait for the kernel before.
-template <typename T, int ITS>
-__global__ void add_norm_vec_kernel(LnArgs a, T* __restrict__ out) {
-    __shared__ float parts[2][LN_MAX_WARPS][3];
-    constexpr bool EARLY = ITS == 1;            // (more sweeps: the weights would not fit beside the rows)
+// hidden % 8 == 0, 8 values per thread and sweep, 16-byte aligned rows: row and delta stay in registers; EARLY: weights are asked
+// for before the wait for the kernel before.
+template <typename T, int ITS, bool EARLY>
+__global__ void __launch_bounds__(512) add_norm_vec_kernel(LnArgs a, T* __restrict__ out) {
+    __shared__ float4 parts[2][LN_MAX_WARPS];
     pdl_launch_dependents();
     const int64_t src = a.rows ? a.rows[blockIdx.x] : blockIdx.x;
     const int H = a.hidden;
     float wd[EARLY ? 8 : 1], w[EARLY ? 8 : 1], bd[EARLY ? 8 : 1];
-    int count = 0;
+    int count = 0, warp_count = 0;              // values of this thread, and of its warp
 #pragma unroll
-    for (int it = 0; it < ITS; ++it) count += (it * (int)blockDim.x + (int)threadIdx.x) * 8 < H ? 8 : 0;
+    for (int it = 0; it < ITS; ++it) {
+        const int at = it * (int)blockDim.x * 8, of_warp = H - at - (int)(threadIdx.x & ~31u) * 8;
+        count += at + (int)threadIdx.x * 8 < H ? 8 : 0;
+        warp_count += min(max(of_warp, 0), 256);
+    }
     if (EARLY && count) {
         ln_load8(a.w + threadIdx.x * 8, w);
         if (a.w_d) ln_load8(a.w_d + threadIdx.x * 8, wd);
@@ -135,7 +130,7 @@ __global__ void add_norm_vec_kernel(LnArgs a, T* __restrict__ out) {
         }
         if (a.w_d) {
             float off, scale;
-            ln_factors(ln_stats(x, count, parts[0], H), a.centred_d, a.eps_d, off, scale);
+            ln_factors(ln_stats(x, count, warp_count, parts[0], H), a.centred_d, a.eps_d, off, scale);
 #pragma unroll
             for (int it = 0; it < ITS; ++it) {
                 const int i = (it * blockDim.x + threadIdx.x) * 8;
@@ -158,7 +153,7 @@ __global__ void add_norm_vec_kernel(LnArgs a, T* __restrict__ out) {
         }
     }
     float off, scale;
-    ln_factors(ln_stats(v, count, parts[1], H), a.centred, a.eps, off, scale);
+    ln_factors(ln_stats(v, count, warp_count, parts[1], H), a.centred, a.eps, off, scale);
 #pragma unroll
     for (int it = 0; it < ITS; ++it) {
         const int i = (it * blockDim.x + threadIdx.x) * 8;
@@ -213,17 +208,23 @@ X0NE_API int x0ne_add_norm(LnArgs a, void* out, int dt, int n_rows, cudaStream_t
     X0NE_REQUIRE(dt == X0NE_F32 || dt == X0NE_BF16, "add_norm: unknown dtype tag %d", dt);
     if (n_rows == 0) return 0;
     const int H = a.hidden;
-    if (H % 8 == 0 && H <= 8 * 1024 * 2 &&
+    if (H % 8 == 0 && H <= 8 * 1024 &&
         ((((uintptr_t)a.resid | (uintptr_t)a.delta | (uintptr_t)a.bias_d | (uintptr_t)a.w_d | (uintptr_t)a.w | (uintptr_t)out) & 15) == 0)) {
         const int pieces = H / 8;
         const bool two = pieces > 512;                      // two sweeps of 512 rather than one of 1,024
         int threads = two ? ((pieces + 1) / 2 + 31) / 32 * 32 : (pieces + 31) / 32 * 32;
-#define LN_VEC(T, ITS) x0ne_launch(add_norm_vec_kernel<T, ITS>, dim3(n_rows), dim3(threads), 0, stream, a, (T*)out)
-        if (dt == X0NE_F32) {
-            if (two) LN_VEC(float, 2); else LN_VEC(float, 1);
-        } else {
-            if (two) LN_VEC(bf16, 2); else LN_VEC(bf16, 1);
-        }
+        // few rows: the weights are asked for before the wait; many rows: fewer registers, so more rows in flight
+        const bool early = !two && n_rows <= 256;
+#define LN_VEC(T, ITS, EARLY) x0ne_launch(add_norm_vec_kernel<T, ITS, EARLY>, dim3(n_rows), dim3(threads), 0, stream, a, (T*)out)
+#define LN_SWEEPS(T)                          \
+    do {                                      \
+        if (two) LN_VEC(T, 2, false);         \
+        else if (early) LN_VEC(T, 1, true);   \
+        else LN_VEC(T, 1, false);             \
+    } while (0)
+        if (dt == X0NE_F32) LN_SWEEPS(float);
+        else LN_SWEEPS(bf16);
+#undef LN_SWEEPS
 #undef LN_VEC
         X0NE_LAUNCH_CHECK();
     }

@@ -139,8 +139,8 @@ class DeltaArg(Structure):
                 ("b_col", c_int32), ("g_col", c_int32), ("conv", c_void_p), ("A", c_void_p), ("dt_bias", c_void_p), ("norm_w", c_void_p),
                 ("q_scale", c_float), ("eps", c_float), ("state", c_void_p), ("state_stride", c_int64), ("ring_off", c_int64),
                 ("row_slot", c_void_p), ("row_pos", c_void_p), ("seq_first_row", c_void_p), ("seq_slot", c_void_p), ("seq_pos0", c_void_p),
-                ("qkv", c_void_p), ("gates", c_void_p), ("o", c_void_p), ("heads", c_int32), ("kv_heads", c_int32), ("D", c_int32), ("V", c_int32),
-                ("taps", c_int32), ("n_rows", c_int32)]
+                ("planes", c_void_p), ("gates", c_void_p), ("o", c_void_p), ("heads", c_int32), ("kv_heads", c_int32), ("D", c_int32), ("V", c_int32),
+                ("taps", c_int32), ("n_rows", c_int32), ("row_len", c_int32)]
 
 
 class AddNormArg(Structure):
@@ -199,7 +199,8 @@ _SIGNATURES = {
     "x0ne_soft_cap": [_P, _L, _F, _P],
     "x0ne_add_norm": [AddNormArg, _P, _I, _I, _P],
     "x0ne_delta_prepare": [DeltaArg, _P],
-    "x0ne_delta_scan": [DeltaArg, _I, _P],
+    "x0ne_delta_scan": [DeltaArg, _I, _P, _P],
+    "x0ne_delta_chunk_scan": [DeltaArg, _P, _I, _I, _P, _P],
     "x0ne_delta_head_norm": [DeltaArg, _P, _I, _L, _P],
     "x0ne_delta_step": [DeltaArg, _P, _I, _L, _I, _P],
     "x0ne_gemm_bf16_smallm_act": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P],
@@ -1115,7 +1116,7 @@ def describe_tc_status(st: int) -> str:
     return (f"a tcgen05 kernel gave up waiting on a barrier (codes {codes}; products: 1 copy, 2 MMA, "
             "3 epilogue, 4 accumulator; attention: 5 queries, 6 keys, 13 and 15 values, 7 probabilities, "
             "8, 11 and 14 output, 10, 12 and 17 scores, 16 and 18 the other half of the row; 9: misaligned "
-            "shared memory); its output is not valid")
+            "shared memory; delta rule: 19 rows of a scan); its output is not valid")
 
 
 def gemm_tc_status(device) -> torch.Tensor:
@@ -1850,6 +1851,13 @@ class DeltaState:
         self.channels = 2 * kv_heads * dim + heads * v_dim
         self.ring_off = -(-heads * v_dim * dim // 4) * 4
         self.floats = -(-(self.ring_off + (taps * self.channels if taps > 1 else 0)) // 4) * 4          # (rows of 16 bytes)
+        # what a row of a pass takes in the planes of prepared q, k and v (delta_rule.cu: dr_row_len, DR_COLS)
+        self.row_len = next((b for b in (32, 64, 128, 256) if dim <= b), -(-dim // 4) * 4) + 8
+        self.plane_floats = 2 * kv_heads * self.row_len + heads * (-(-v_dim // 16) * 16)
+
+    def chunks_take(self) -> bool:
+        """Whether the scan by chunks takes these widths."""
+        return self.dim <= DELTA_STEP_MAX_DIM
 
     def step_takes(self) -> bool:
         """Whether the one-launch kernel for passes of one token per sequence takes these widths."""
@@ -1858,12 +1866,13 @@ class DeltaState:
 
 def delta_arg(g: DeltaState, src: torch.Tensor, cols, conv: torch.Tensor, A: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor, q_scale: float,
               eps: float, state: torch.Tensor, row_slot: torch.Tensor, row_pos: torch.Tensor, seq_first_row: torch.Tensor, seq_slot: torch.Tensor,
-              seq_pos0: torch.Tensor, n_rows: int, qkv: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None,
+              seq_pos0: torch.Tensor, n_rows: int, planes: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None,
               o: Optional[torch.Tensor] = None) -> DeltaArg:
     """What the delta rule's kernels read and write.  `src`: the float32 projection; `cols`: where q, k, v, a, b and the output
-    gate start in its rows; `conv` [channels, taps]: q's channels, k's, v's; qkv, gates, o: buffers for passes of many tokens."""
+    gate start in its rows; `conv` [channels, taps]: q's channels, k's, v's; planes, gates, o: buffers for passes of many tokens
+    (n_rows x plane_floats, 4 heads and heads * v_dim values)."""
     for t, what in ((src, "projection"), (conv, "convolution taps"), (A, "decay rates"), (dt_bias, "decay biases"), (norm_w, "head norm weight"), (state, "state"),
-                    (qkv, "prepared rows"), (gates, "gates"), (o, "scan output")):
+                    (planes, "prepared rows"), (gates, "gates"), (o, "scan output")):
         if t is not None:
             _need(t, torch.float32, what)
     hv = g.heads * g.v_dim
@@ -1871,24 +1880,43 @@ def delta_arg(g: DeltaState, src: torch.Tensor, cols, conv: torch.Tensor, A: tor
     if max(ends) > src.shape[-1] or src.numel() < n_rows * src.shape[-1] or tuple(conv.shape) != (g.channels, g.taps) or A.numel() != g.heads \
             or dt_bias.numel() != g.heads or norm_w.numel() != g.v_dim or state.dim() != 2 or state.shape[1] < g.floats:
         raise KernelError("delta rule: shapes do not match")
-    for t, width in ((qkv, g.channels), (gates, 2 * g.heads), (o, hv)):
+    for t, width in ((planes, g.plane_floats), (gates, 4 * g.heads), (o, hv)):
         if t is not None and (t.shape[-1] != width or t.numel() < n_rows * width):
             raise KernelError("delta rule: a buffer does not match the heads or rows")
     return DeltaArg(_ptr(src), src.shape[-1], *cols, _ptr(conv), _ptr(A), _ptr(dt_bias), _ptr(norm_w), float(q_scale), float(eps), _ptr(state), state.stride(0),
-                    g.ring_off, _ptr(row_slot), _ptr(row_pos), _ptr(seq_first_row), _ptr(seq_slot), _ptr(seq_pos0), _ptr(qkv), _ptr(gates), _ptr(o), g.heads,
-                    g.kv_heads, g.dim, g.v_dim, g.taps, n_rows)
+                    g.ring_off, _ptr(row_slot), _ptr(row_pos), _ptr(seq_first_row), _ptr(seq_slot), _ptr(seq_pos0), _ptr(planes), _ptr(gates), _ptr(o), g.heads,
+                    g.kv_heads, g.dim, g.v_dim, g.taps, n_rows, g.row_len)
 
 
 def delta_prepare(a: DeltaArg) -> None:
-    """Convolution, activation and unit vectors of every row's q, k and v into qkv, decays and write strengths into gates."""
+    """Convolution, activation and unit vectors of every row's q, k and v into the planes, decays and write strengths into gates."""
     lib = _lib("core")
     _check(lib, lib.x0ne_delta_prepare(a, _stream()), "delta_prepare")
 
 
 def delta_scan(a: DeltaArg, n_seqs: int) -> None:
-    """Token by token over every sequence's prepared rows, from and into its state; the convolutions' inputs join the state."""
+    """Token by token over every sequence's prepared rows, from and into its state; the convolutions' inputs join the state.  A
+    wait for copies that ran out shows in `gemm_tc_status`."""
+    global tc_used
     lib = _lib("core")
-    _check(lib, lib.x0ne_delta_scan(a, n_seqs, _stream()), "delta_scan")
+    tc_used = True
+    _check(lib, lib.x0ne_delta_scan(a, n_seqs, _ptr(gemm_tc_status(torch.device("cuda", torch.cuda.current_device()))), _stream()), "delta_scan")
+
+
+DELTA_CHUNK, DELTA_COEF = 8, 20
+
+
+def delta_chunk_scan(a: DeltaArg, coef: torch.Tensor, n_seqs: int, max_seq_rows: int) -> None:
+    """The scan by chunks of DELTA_CHUNK tokens, in two launches: the same rule with the products between a chunk's tokens worked out
+    ahead (into `coef`, float32 [rows, heads * DELTA_COEF]); results equal delta_scan's to rounding.  Heads of up to 256 channels."""
+    lib = _lib("core")
+    _need(coef, torch.float32, "chunk coefficients")
+    if coef.shape[-1] != a.heads * DELTA_COEF or coef.numel() < a.n_rows * coef.shape[-1]:
+        raise KernelError("delta_chunk_scan: the coefficients' buffer does not match the heads or rows")
+    global tc_used, LAUNCHES
+    tc_used = True
+    _check(lib, lib.x0ne_delta_chunk_scan(a, _ptr(coef), n_seqs, max_seq_rows, _ptr(gemm_tc_status(coef.device)), _stream()), "delta_chunk_scan")
+    LAUNCHES += 1
 
 
 def _delta_out(a: DeltaArg, out: torch.Tensor) -> None:

@@ -74,7 +74,7 @@ class GatedDeltaRule(ProjectedMixer):
         ws, rows, g = ctx.ws, ctx.ws.max_rows, self.geometry
         state = ctx.cache.state(entry, self.tag)
         one = ctx.decode and g.step_takes()
-        buffers = {} if one else dict(qkv=ws.buffer("delta.qkv", (rows, g.channels), torch.float32), gates=ws.buffer("delta.gates", (rows, 2 * g.heads), torch.float32),
+        buffers = {} if one else dict(planes=ws.buffer("delta.planes", (rows, g.plane_floats), torch.float32), gates=ws.buffer("delta.gates", (rows, 4 * g.heads), torch.float32),
                                       o=ws.buffer("delta.o", (rows, self.out_dim), torch.float32))
         a = ops.delta_arg(g, proj, [col + c for c in self.cols], self.conv, self.A, self.dt_bias, self.norm, g.dim ** -0.5, self.eps, state, ctx.row_slot,
                           ctx.row_pos, ctx.seq_first_row, ctx.seq_slot, ctx.seq_pos0, n_rows, **buffers)
@@ -82,7 +82,11 @@ class GatedDeltaRule(ProjectedMixer):
             ops.delta_step(a, act, ctx.n_seqs)
         else:
             ops.delta_prepare(a)
-            ops.delta_scan(a, ctx.n_seqs)
+            # 32-bit runs walk token by token, so that a token's bits do not depend on where its pass began
+            if self.env.dtype == torch.bfloat16 and ctx.max_seq_rows >= ops.DELTA_CHUNK and g.chunks_take():
+                ops.delta_chunk_scan(a, ws.buffer("delta.coef", (rows, g.heads * ops.DELTA_COEF), torch.float32), ctx.n_seqs, ctx.max_seq_rows)
+            else:
+                ops.delta_scan(a, ctx.n_seqs)
             ops.delta_head_norm(a, act)
 
 
