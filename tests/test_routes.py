@@ -37,13 +37,22 @@ def test_every_row_count_of_every_shape_has_a_rule_and_every_rule_is_reached():
     reached = set()
     shapes = [(n, k) for size in SIZES for n, k in matrices(size).values()] + [(64, 64), (160, 96), (151936, 4096), (8, 8)]
     for n, k in shapes:
-        for fused in (False, True):
+        for fused, act in ((False, False), (True, False), (False, True)):
             for rows in list(range(1, 130)) + [767, 768, 5000, 1 << 20]:
-                rule = routes.choose(rows, n, k, fused=fused)
+                rule = routes.choose(rows, n, k, fused=fused, act=act)
                 assert rule.kernel in ("smallm", "skinny", "tc_pair", "library") and rule.why
                 reached.add(id(rule))
     assert len(reached) == len(routes.RULES)
     assert routes.RULES[-1].kernel == "library" and routes.RULES[-1].rows == (1, 1 << 30) and routes.RULES[-1].fused is None
+
+
+@pytest.mark.parametrize("n,k,rows,expect", [
+    (9216, 2048, 8, "smallm"), (9216, 2048, 32, "skinny"), (9216, 2048, 64, "skinny"), (9216, 2048, 128, "library"), (9216, 2048, 2048, "tc_pair"),
+    (18432, 4096, 64, "skinny"), (18432, 4096, 2048, "library"),
+])
+def test_products_with_an_activation_behind_them(n, k, rows, expect):
+    assert routes.kernel_for(rows, n, k, act=True) == expect
+    assert routes.kernel_for(rows, n, k) in ("smallm", "skinny", "library")          # (the rules of an activation are its own)
 
 
 def test_fill_of_the_weight_streaming_kernel():

@@ -426,6 +426,32 @@ def test_heads_side_by_side_times_their_gate(heads, vd, dtype):
     assert (out.double() - want).abs().max() <= (1e-6 if dtype == "float32" else 2 ** -8) * want.abs().max()
 
 
+@pytest.mark.parametrize("rows", [1, 5, 8, 9, 32])
+@pytest.mark.parametrize("heads,k,n,rot,half", [(5, 12, 22, 8, True), (3, 128, 70, 32, False), (2, 200, 33, 0, True), (4, 260, 128, 16, True), (1, 1000, 5, 0, False)])
+def test_products_per_head_of_few_rows(heads, k, n, rot, half, rows):
+    from x0ne_engine_b200.csrc import ops
+    g = torch.Generator().manual_seed(k + rows)
+    r = lambda *s: torch.randn(*s, generator=g).bfloat16()
+    x, w, gate = r(rows, heads * (k + rot) + 4), r(heads, n, k), r(rows, heads * n + 9)
+    pos = [7 + 13 * i for i in range(rows)]
+    xh = x[:, :heads * (k + rot)].double().view(rows, heads, k + rot)
+    y = torch.einsum("hnk,rhk->rhn", w.double(), xh[..., :k])
+    xd, wd, gd = x.to(DEV), w.to(DEV), gate.to(DEV)
+    assert ops.head_products_take(xd, x.shape[1], k + rot, wd, rows)
+    out = torch.full((rows, heads * n), 7.0, dtype=torch.bfloat16, device=DEV)
+    ops.head_products(xd, x.shape[1], k + rot, wd, out, n, rows, gate=gd[0, 3:], gate_ld=heads * n + 9)
+    want = y.reshape(rows, -1) * torch.sigmoid(gate[:, 3:3 + heads * n].double())
+    assert (out.double().cpu() - want).abs().max() <= 2 ** -8 * want.abs().max()
+    freq = torch.tensor(P.yarn(rot, 70.0, None)[0], dtype=torch.float32, device=DEV) if rot else None
+    out = torch.full((rows, heads * (n + rot)), 7.0, dtype=torch.bfloat16, device=DEV)
+    ops.head_products(xd, x.shape[1], k + rot, wd, out, n + rot, rows, turn=ops.latent_turn(freq, None, 1.25, rot, half), row_pos=i32(pos))
+    tail = xh[..., k:].contiguous()
+    if rot:
+        tail = 1.25 * P.rotate(tail, torch.tensor(pos), {"dims": rot, "base": 70.0}, "half" if half else "interleaved")
+    want = torch.cat([y, tail], dim=-1).reshape(rows, -1)
+    assert (out.double().cpu() - want).abs().max() <= 2 ** -7 * want.abs().max()
+
+
 # ------------------------------------------------------------------------------------------ activations in the products
 @pytest.mark.parametrize("m", [1, 8, 12, 40, 64, 300, 1000])
 @pytest.mark.parametrize("n,k", [(176, 128), (1000, 512), (8192, 256)])

@@ -643,10 +643,10 @@ def cmd_kernel_bench(a) -> int:
                 raise SystemExit("delta_step takes one row per sequence: --m 1")
             timed(lambda: ops.delta_step(arg, act, B), rows * (g.channels * (1 + 2 * taps) * 4 + hv * (4 + 2)) + states, flops)
         return 0
-    if a.kernel in ("add_norm", "heads_gate", "latent_rows", "latent_queries"):
+    if a.kernel in ("add_norm", "heads_gate", "latent_rows", "latent_queries", "head_products"):
         # --m rows: the add of a pending result that is layer-normed first and the layer norm of the sum (--n values); the heads of a
         # product per head gated and laid side by side (--q-heads x --v-dim); latent attention's rows and queries (--latent-rank
-        # latents, query latents of --n, a rotated part of 64)
+        # latents, query latents of --n, a rotated part of 64); the same queries carried into the latent space and turned in one launch
         from .cache import SequenceCache
         from .parts.base import CacheNeed
         rows, h, heads, d, rank, rot = a.m, a.n, a.q_heads, a.head_dim, a.latent_rank or 256, 64
@@ -672,6 +672,11 @@ def cmd_kernel_bench(a) -> int:
             src, cq = bf(rows, h + rank + rot), torch.empty(rows, h, device=dev, dtype=torch.bfloat16)
             wq, wkv = torch.ones(h, device=dev), torch.ones(rank, device=dev)
             timed(lambda: ops.latent_rows(src, 0, h, wq, cq, h, rank, wkv, 1e-6, turn, cache.kv_view(0), slots, pos, rows), rows * (h + rank + rot) * 4)
+            return 0
+        if a.kernel == "head_products":
+            q, w, out = bf(rows, heads * (d + rot)), bf(heads, rank, d), bf(rows, heads * (rank + rot))
+            timed(lambda: ops.head_products(q, heads * (d + rot), d + rot, w, out, rank + rot, rows, turn=turn, row_pos=pos),
+                  (w.numel() + q.numel() + out.numel()) * 2)
             return 0
         q, q_abs = bf(rows, heads * (d + rot)), bf(heads, rows, rank)
         out = torch.empty(rows, heads * (rank + rot), device=dev, dtype=torch.bfloat16)

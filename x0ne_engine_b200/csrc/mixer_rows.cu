@@ -1387,6 +1387,135 @@ X0NE_API int x0ne_heads_gate(const void* x, int64_t head_stride, const void* gat
 }
 
 // ----------------------------------------------------------------------------------------
+// A product per head for few rows, bfloat16 with float32 sums:  y[row][h][n] = sum_k W[h][n][k] x[row][h][k], and what follows it:
+//   gate given:  out = y * sigmoid(gate[row * gate_ld + h * N + n])
+//   turn.rot > 0: out is y, and behind a head's N values the head's `rot` turned ones, taken from behind its K values of x
+// Row r, head h of x starts at r * x_ld + h * x_head, of out at r * out_ld + h * out_head.  A warp takes four outputs; its weights are
+// asked for before the wait for the kernel before; every lane has pieces of four inner values; the 4 outputs x 8 rows of a pass over
+// the rows are summed over the lanes together, each lane ending up with one of them.
+// ----------------------------------------------------------------------------------------
+struct HeadProductArgs {
+    const bf16* x;
+    int64_t x_ld;
+    int32_t x_head;
+    const bf16* w;              // [heads][N][K]
+    bf16* out;
+    int64_t out_ld;
+    int32_t out_head;
+    const bf16* gate;
+    int64_t gate_ld;
+    LatentTurn turn;
+    const int32_t* row_pos;
+    int32_t n_rows, heads, N, K;
+};
+#define HP_ROWS 8
+#define HP_OUT 4
+#define HP_WARPS 4
+
+template <int PIECES>
+__global__ void __launch_bounds__(HP_WARPS * 32) head_products_kernel(HeadProductArgs a) {
+    extern __shared__ __align__(16) float hp_x[];           // [HP_ROWS][K]
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x;
+    const int n0 = (blockIdx.y * HP_WARPS + warp) * HP_OUT, K = a.K;
+    const int n_blocks = (a.N + HP_WARPS * HP_OUT - 1) / (HP_WARPS * HP_OUT);
+    if ((int)blockIdx.y == n_blocks) {                      // the turned values
+        const int half = a.turn.rot / 2;
+        pdl_wait();
+        for (int i = tid; i < a.n_rows * half; i += HP_WARPS * 32) {
+            const int row = i / half, j = i - row * half;
+            float c, sn;
+            latent_turn(a.turn, a.row_pos[row], j, c, sn);
+            const int iu = a.turn.half_layout ? j : 2 * j, iv = a.turn.half_layout ? j + half : 2 * j + 1;
+            const bf16* from = a.x + (int64_t)row * a.x_ld + (int64_t)h * a.x_head + K;
+            bf16* to = a.out + (int64_t)row * a.out_ld + (int64_t)h * a.out_head + a.N;
+            const float u = to_f32(from[iu]), v = to_f32(from[iv]);
+            to[iu] = from_f32<bf16>(u * c - v * sn);
+            to[iv] = from_f32<bf16>(v * c + u * sn);
+        }
+        return;
+    }
+    uint2 w[HP_OUT][PIECES];
+#pragma unroll
+    for (int o = 0; o < HP_OUT; ++o)
+#pragma unroll
+        for (int p = 0; p < PIECES; ++p) {
+            const int k = (p * 32 + lane) * 4;
+            w[o][p] = make_uint2(0u, 0u);
+            if (k < K && n0 + o < a.N) w[o][p] = *reinterpret_cast<const uint2*>(a.w + ((int64_t)h * a.N + n0 + o) * K + k);
+        }
+    pdl_wait();
+    for (int r0 = 0; r0 < a.n_rows; r0 += HP_ROWS) {
+        const int nr = min(HP_ROWS, a.n_rows - r0);
+        __syncthreads();
+        for (int i = tid; i < HP_ROWS * (K / 4); i += HP_WARPS * 32) {
+            const int r = i / (K / 4), k = (i - r * (K / 4)) * 4;
+            uint2 x = make_uint2(0u, 0u);
+            if (r < nr) x = *reinterpret_cast<const uint2*>(a.x + (int64_t)(r0 + r) * a.x_ld + (int64_t)h * a.x_head + k);
+            const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
+            *reinterpret_cast<float4*>(hp_x + r * K + k) = make_float4(lo.x, lo.y, hi.x, hi.y);
+        }
+        __syncthreads();
+        float acc[HP_OUT * HP_ROWS];
+#pragma unroll
+        for (int e = 0; e < HP_OUT * HP_ROWS; ++e) acc[e] = 0.f;
+#pragma unroll
+        for (int p = 0; p < PIECES; ++p) {
+            const int k = (p * 32 + lane) * 4;
+            if (k >= K) break;
+            float4 wf[HP_OUT];
+#pragma unroll
+            for (int o = 0; o < HP_OUT; ++o) {
+                const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[o][p].x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[o][p].y));
+                wf[o] = make_float4(lo.x, lo.y, hi.x, hi.y);
+            }
+#pragma unroll
+            for (int r = 0; r < HP_ROWS; ++r) {
+                const float4 x = *reinterpret_cast<const float4*>(hp_x + r * K + k);
+#pragma unroll
+                for (int o = 0; o < HP_OUT; ++o) {
+                    float& s = acc[o * HP_ROWS + r];
+                    s = fmaf(wf[o].x, x.x, s); s = fmaf(wf[o].y, x.y, s); s = fmaf(wf[o].z, x.z, s); s = fmaf(wf[o].w, x.w, s);
+                }
+            }
+        }
+        // 32 values over 32 lanes: lane l ends up with the sum of value l
+#pragma unroll
+        for (int off = 16; off >= 1; off >>= 1) {
+            const bool up = (lane & off) != 0;
+#pragma unroll
+            for (int i = 0; i < off; ++i) {
+                const float mine = up ? acc[i + off] : acc[i], other = up ? acc[i] : acc[i + off];
+                acc[i] = mine + __shfl_xor_sync(0xffffffffu, other, off);
+            }
+        }
+        const int r = lane % HP_ROWS, n = n0 + lane / HP_ROWS;
+        if (r < nr && n < a.N) {
+            float y = acc[0];
+            if (a.gate != nullptr) y /= 1.0f + expf(-to_f32(a.gate[(int64_t)(r0 + r) * a.gate_ld + (int64_t)h * a.N + n]));
+            a.out[(int64_t)(r0 + r) * a.out_ld + (int64_t)h * a.out_head + n] = from_f32<bf16>(y);
+        }
+    }
+}
+
+X0NE_API int x0ne_head_products(HeadProductArgs a, cudaStream_t stream) {
+    X0NE_REQUIRE(a.n_rows >= 0 && a.heads > 0 && a.N > 0 && a.K > 0 && a.K % 4 == 0 && a.K <= 1024 && a.x != nullptr && a.w != nullptr && a.out != nullptr,
+                 "head_products: rows %d, %d heads of %d x %d", a.n_rows, a.heads, a.N, a.K);
+    X0NE_REQUIRE(a.turn.rot >= 0 && a.turn.rot % 2 == 0 && (a.turn.rot == 0 || (a.turn.freq != nullptr && a.row_pos != nullptr && a.gate == nullptr && a.x_head >= a.K + a.turn.rot &&
+                                                                             a.out_head >= a.N + a.turn.rot)), "head_products: %d turned values", a.turn.rot);
+    X0NE_REQUIRE(a.x_head >= a.K && a.out_head >= a.N && a.x_ld % 4 == 0 && a.x_head % 4 == 0 && ((((uintptr_t)a.x | (uintptr_t)a.w) & 7) == 0), "head_products: rows are not 8-byte aligned");
+    if (a.n_rows == 0) return 0;
+    const dim3 grid(a.heads, (a.N + HP_WARPS * HP_OUT - 1) / (HP_WARPS * HP_OUT) + (a.turn.rot > 0 ? 1 : 0)), block(HP_WARPS * 32);
+    const size_t smem = (size_t)HP_ROWS * a.K * sizeof(float);
+    const int pieces = (a.K + 127) / 128;
+    if (pieces <= 1) x0ne_launch(head_products_kernel<1>, grid, block, smem, stream, a);
+    else if (pieces <= 2) x0ne_launch(head_products_kernel<2>, grid, block, smem, stream, a);
+    else if (pieces <= 4) x0ne_launch(head_products_kernel<4>, grid, block, smem, stream, a);
+    else x0ne_launch(head_products_kernel<8>, grid, block, smem, stream, a);
+    X0NE_LAUNCH_CHECK();
+}
+
+// ----------------------------------------------------------------------------------------
 // x = cap tanh(x / cap) in place, float32.
 // ----------------------------------------------------------------------------------------
 __global__ void soft_cap_kernel(float* __restrict__ x, int64_t total, float cap) {

@@ -161,6 +161,13 @@ class LatentRowsArg(Structure):
                 ("row_pos", c_void_p), ("n_rows", c_int32), ("write_cache", c_int32)]
 
 
+class HeadProductArg(Structure):
+    """Mirror of `struct HeadProductArgs` in mixer_rows.cu."""
+    _fields_ = [("x", c_void_p), ("x_ld", c_int64), ("x_head", c_int32), ("w", c_void_p), ("out", c_void_p), ("out_ld", c_int64), ("out_head", c_int32),
+                ("gate", c_void_p), ("gate_ld", c_int64), ("turn", LatentTurnArg), ("row_pos", c_void_p), ("n_rows", c_int32), ("heads", c_int32),
+                ("N", c_int32), ("K", c_int32)]
+
+
 class SampleIOArg(Structure):
     """Mirror of `struct SampleIO` in sampling.cu."""
     _fields_ = [("logits", c_void_p), ("temperature", c_void_p), ("top_p", c_void_p), ("seed", c_void_p),
@@ -195,6 +202,7 @@ _SIGNATURES = {
     "x0ne_rope_pairs_kv_write": [_P, _P, _I, _I, _I, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _I, _I, None, _P, _P, _I, _I, _P],
     "x0ne_latent_rows": [LatentRowsArg, _P, _I, None, _P],
     "x0ne_latent_queries": [_P, _L, _P, _L, LatentTurnArg, _P, _P, _I, _I, _I, _I, _I, _P],
+    "x0ne_head_products": [HeadProductArg, _P],
     "x0ne_heads_gate": [_P, _L, _P, _L, _P, _I, _I, _I, _I, _P],
     "x0ne_soft_cap": [_P, _L, _F, _P],
     "x0ne_add_norm": [AddNormArg, _P, _I, _I, _P],
@@ -1835,6 +1843,32 @@ def heads_gate(x: torch.Tensor, gate: torch.Tensor, gate_ld: int, out: torch.Ten
         raise KernelError("heads_gate: shapes or types do not match")
     _check(lib, lib.x0ne_heads_gate(_ptr(x), x.stride(0), _ptr(gate), gate_ld, _ptr(out), dtype_tag(out.dtype), n_rows, x.shape[0], x.shape[2], _stream()),
            "heads_gate")
+
+
+HEAD_PRODUCT_MAX_ROWS = 32       # passes of at most this many rows give a product per head to head_products
+
+
+def head_products_take(x: torch.Tensor, x_ld: int, x_head: int, w: torch.Tensor, n_rows: int) -> bool:
+    """Whether head_products takes this product per head ([heads, N, K] weights against n_rows rows of `x`)."""
+    return x.dtype == torch.bfloat16 and n_rows <= HEAD_PRODUCT_MAX_ROWS and w.shape[2] % 4 == 0 and w.shape[2] <= 1024 and x_ld % 4 == 0 and x_head % 4 == 0
+
+
+def head_products(x: torch.Tensor, x_ld: int, x_head: int, w: torch.Tensor, out: torch.Tensor, out_head: int, n_rows: int, gate: Optional[torch.Tensor] = None,
+                  gate_ld: int = 0, turn: Optional[LatentTurnArg] = None, row_pos: Optional[torch.Tensor] = None) -> None:
+    """out[row, h] = w[h] x[row, h] (bfloat16, float32 sums, few rows) with x's row r, head h at r * x_ld + h * x_head: times
+    sigmoid(gate[row, h]) with `gate` (a view whose rows start gate_ld values apart, a value per output), or with the head's turned values
+    behind it (`turn`, `row_pos`), taken from behind its K values of x."""
+    lib = _lib("core")
+    _need(w, torch.bfloat16, "weights per head")
+    _need(out, torch.bfloat16, "output")
+    heads, n, k = w.shape
+    if x.dtype != torch.bfloat16 or not x.is_cuda or (gate is not None and (gate.dtype != torch.bfloat16 or not gate.is_cuda)):
+        raise KernelError("head_products: rows and gates are bfloat16 on the GPU")
+    if x.numel() < (n_rows - 1) * x_ld + (heads - 1) * x_head + k or out.shape[-1] < heads * out_head or out.numel() < n_rows * out.shape[-1]:
+        raise KernelError("head_products: buffers smaller than the rows asked for")
+    arg = HeadProductArg(_ptr(x), x_ld, x_head, _ptr(w), _ptr(out), out.shape[-1], out_head, _ptr(gate), gate_ld,
+                         turn if turn is not None else LatentTurnArg(None, None, 1.0, 0, 0, 0), _ptr(row_pos), n_rows, heads, n, k)
+    _check(lib, lib.x0ne_head_products(arg, _stream()), "head_products")
 
 
 DELTA_STEP_MAX_DIM, DELTA_STEP_MAX_VALUES, DELTA_MAX_TAPS = 256, 2048, 64

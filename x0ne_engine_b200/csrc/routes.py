@@ -86,12 +86,18 @@ RULES: List[Rule] = [
          "gate|up 24576 x 4096 at 32 rows: skinny 36.2 us, library 36.7 + the SwiGLU launch; at 64: 38.1 = 38.1 + the launch"),
     Rule("skinny", (17, 64), False, lambda s: s.long_rows and s.weight_bytes >= 2 * MB,
          "4096 x 12288 at 64 rows: skinny 20.8 us, library 21.8; 5120 x 25600: 44.3 / 46.8; 2048 x 6144: 10.2 / 10.6"),
+    Rule("skinny", (17, 64), False, lambda s: s.weight_bytes >= 2 * MB,
+         "squared ReLU behind 9216 x 2048 at 64 rows: skinny 10.3 us with it in the epilogue, library 14.8 + its launch; "
+         "18432 x 4096: 32.6 against 33.6 in all; 6144 x 2048: 11.4 / 14.9", act=True),
     Rule("skinny", (17, 48), False, lambda s: s.weight_bytes >= 64 * MB,
          "10240 x 5120 at 32 rows: skinny 20.1 us, library 21.1; 5120 x 8192: 17.0 / 19.4; at 64 rows the library is ahead on both"),
     # ---- many rows
     Rule("library", (768, 2048), True, lambda s: s.k <= 2048,
          "gate|up 12288 x 2048 at 2,048 rows: library 89.8 us with the activation's launch, tc_pair 99.9 (113.1 with biases in the "
          "epilogue: a tile of 32 steps over K does not cover it)"),
+    Rule("tc_pair", (1536, 1 << 30), False, lambda s: s.k <= 2048 and s.n >= 2 * s.k,
+         "squared ReLU behind 9216 x 2048 at 2,048 rows: 56.6 us in the epilogue, library 59.8 with the launch; 6144 x 2048: 56.5 / 60.7 "
+         "(at 4,096: 82.5 / 114.9); 18432 x 4096 stays with the library, 213.7 against 220.6", act=True),
     Rule("tc_pair", (768, 1 << 30), True, _always,
          "gate|up 24576 x 4096 at 2,048 rows: 1.62 PFLOP/s with the activation in the epilogue; at 512 rows the library "
          "(74.9 us + 8.5 for SwiGLU) is ahead of it (84.6)"),

@@ -125,9 +125,12 @@ class LatentAttention(Mixer):
                 q, q_ld = ctx.ws.buffer("lattn.q_heads", (rows, self.q_width), dt), self.q_width
                 self.uq(cq, q, n_rows)
         # queries into the latent space, head by head: q_abs[h] = q[:, h, :head_dim] K_h
-        q_un = q[:n_rows, :self.q_width].view(n_rows, H, d + r)[:, :, :d].permute(1, 0, 2)
-        ops.batched_product(q_un, self.uk_t, q_abs)
-        if self.one_launch:
+        few = not self.one_launch and ops.head_products_take(q, q_ld, d + r, self.uk_t, n_rows)         # (one launch with what follows the product)
+        if not few:
+            ops.batched_product(q[:n_rows, :self.q_width].view(n_rows, H, d + r)[:, :, :d].permute(1, 0, 2), self.uk_t, q_abs)
+        if few:
+            ops.head_products(q, q_ld, d + r, self.uk_t, q_full, rank + r, n_rows, turn=turn, row_pos=ctx.row_pos)
+        elif self.one_launch:
             ops.latent_prepare(proj, self.cols[1], q_abs, self.norm_w, self.eps, freq, mag, table, q_full, H, d, r, rank, view, ctx.row_slot,
                                ctx.row_pos, n_rows, write_cache)
         else:
@@ -137,7 +140,9 @@ class LatentAttention(Mixer):
         run_attention_ex(ctx, q_full, o_lat, view, n_rows, H, self.scale, self.window, extra)
         # back out of the latent space: head h's values are V_h (weights . c)
         o_heads = o_lat[:n_rows].view(n_rows, H, rank).permute(1, 0, 2)
-        if self.has_gate and self.gate_wide:
+        if self.has_gate and self.gate_wide and ops.head_products_take(o_lat, H * rank, rank, self.uv, n_rows):
+            ops.head_products(o_lat, H * rank, rank, self.uv, att, vd, n_rows, gate=gate, gate_ld=width)
+        elif self.has_gate and self.gate_wide:
             v_heads = ctx.ws.buffer("lattn.v_heads", (H * rows * vd,), dt)[:H * n_rows * vd].view(H, n_rows, vd)
             ops.batched_product(o_heads, self.uv, v_heads)
             ops.heads_gate(v_heads, gate, width, att, n_rows)
